@@ -582,7 +582,7 @@ int lp_parity_softmax(float* scores, long long ld, int Tq, int Tk, float scale, 
  * mechanisms are separate entry points with their constants as arguments, so that a model description (a list of layers) composes
  * them: csrc/lp_linear.cu, lp_stream32.cu, lp_seqmix.cu, lp_moe.cu.
  * ------------------------------------------------------------------------------------------------------------------ */
-enum lp_linear_epi { LP_EPI_NONE = 0, LP_EPI_XIELU = 1, LP_EPI_SILU_GATE = 2, LP_EPI_RELU2 = 3, LP_EPI_CLAMP_GLU = 4 };
+enum lp_linear_epi { LP_EPI_NONE = 0, LP_EPI_XIELU = 1, LP_EPI_SILU_GATE = 2, LP_EPI_RELU2 = 3, LP_EPI_CLAMP_GLU = 4, LP_EPI_GELU_GATE = 5 };
 enum lp_rot_layout { LP_ROT_HALF = 0, LP_ROT_INTERLEAVED = 1 };
 #define LP_RETENTION_CHUNK 32
 #define LP_LATENT_SPLIT_ROWS 16   /* lp_latent_attend: up to this many rows a CTA per (row, head) splits the keys over its warps */
@@ -591,9 +591,11 @@ enum lp_rot_layout { LP_ROT_HALF = 0, LP_ROT_INTERLEAVED = 1 };
  * bf16.  epi XIELU: a z^2 + z/2 (z > 0), b (exp(z) - 1 - z) + z/2 (z <= 0) with a = epi_a, b = epi_b.  epi SILU_GATE: W = [gate rows;
  * up rows], N' = N / 2, C = silu(gate) * up.  epi RELU2: max(z, 0)^2.  fp32 FMA accumulation in K order.  c_accum != 0: the result
  * is not stored but added, C <- C + c_scale * epi(...) (x <- x + m * sublayer(x) in the product's own store).
+ * epi GELU_GATE: the same with C = gelu(gate) * up, gelu in its tanh form.
  * epi CLAMP_GLU: W = [gate rows; up rows], N' = N / 2, g = min(gate, epi_a), u = clamp(up, -epi_a, epi_a), C = g sigmoid(epi_b g) (u + 1).
  * Before the epilogue an accumulator becomes row_scale[m] * acc + bias[n] (either may be NULL; m is the row of C, for lp_linear_pairs
- * the pair; one problem only).  gate (fp32 [rows of C, ldg], or NULL): the epilogue's result is multiplied by sigmoid(gate[m, n]). */
+ * the pair; one problem only).  gate (fp32 [rows of C, ldg], or NULL): the epilogue's result is multiplied by sigmoid(gate[m, n]);
+ * problem z of a batch reads gate + z * gate_batch. */
 typedef struct lp_linear_desc {
   const void* A; long long lda; long long a_batch; int a_fp32;
   const void* W; long long ldw; long long w_batch;
@@ -602,7 +604,7 @@ typedef struct lp_linear_desc {
   int epi; float epi_a, epi_b;
   int c_accum; float c_scale;
   const float* bias; const float* row_scale;
-  const float* gate; long long ldg;
+  const float* gate; long long ldg; long long gate_batch;
 } lp_linear_desc;
 int lp_linear(const lp_linear_desc* desc, void* stream);
 /* row tiles of lp_linear_tile_rows() rows, each multiplied by the weight of group tile_group[tile] (w_batch elements apart; < 0: the
@@ -618,8 +620,8 @@ int lp_embed_rows_f32(const int* ids, int R, const void* table, long long ldt, i
 /* y = x / sqrt(mean(x^2) + eps) * gain_scalar (* gain_vec[c]); written to `out` (fp32 or bf16) or added to `accum` (fp32) */
 int lp_rmsnorm_f32(const float* x, long long ldx, int M, int D, float gain_scalar, const float* gain_vec, float eps, void* out,
                    long long ldo, int out_fp32, float* accum, long long ld_accum, void* stream);
-/* standalone activation for products that ran on lp_gemm_bf16: mode XIELU, RELU2 (N columns) or SILU_GATE, CLAMP_GLU (in has 2N
- * columns: gate | up) */
+/* standalone activation for products that ran on lp_gemm_bf16: mode XIELU, RELU2 (N columns) or SILU_GATE, GELU_GATE, CLAMP_GLU
+ * (in has 2N columns: gate | up) */
 int lp_glu_f32(const void* in, long long ldi, int in_fp32, void* out, long long ldo, int out_fp32, int M, int N, int mode, float a,
                float b, void* stream);
 /* the same with every input of row m first multiplied by row_scale[m] (NULL: 1) */
@@ -671,7 +673,8 @@ int lp_retention_decode(const lp_retention_desc* desc, int n_seqs, const int* se
 /* Latent attention over a paged cache of rows [c (kv_rank) | rotated shared key (rot_dim)] fp32; page_table int32 [requests, max_pages]. */
 typedef struct lp_latent_desc {
   float* q; long long ldq;                  /* [rows, heads * (dim + rot_dim)]: per head [unrotated | rotated] */
-  const float* dkv; long long lddkv;        /* [rows, kv_rank + rot_dim] (lp_latent_prep only) */
+  const float* dkv; long long lddkv;        /* [rows, kv_rank + rot_dim] (lp_latent_prep only); NULL: `cache` is another layer's, already
+                                               written for this step's rows, and lp_latent_prep rotates the queries only */
   int heads, dim, rot_dim, kv_rank;
   const float* c_gain; float eps;           /* RMS norm of the latent: vector gain */
   const float* inv_freq; int rot_dims; int rot_layout; float rot_mscale;
@@ -695,7 +698,9 @@ int lp_latent_attend(const lp_latent_desc* desc, int R, const int* row_seq, cons
  *   - with pool = P > 0: one key / value per block of P tokens that lies wholly before the window (block b = positions bP .. bP+P-1
  *     is seen when bP + P - 1 <= i - window); they are the means of the block's cached key and value rows, kept in a second paged
  *     pool `pooled` with one row per block (pooled_table: pages of block rows per request).
- * score = q . k * scale, then softcap * tanh(score / softcap) when softcap > 0.  One softmax over everything visible; sink != 0 adds
+ * score = q . k * scale, then softcap * tanh(score / softcap) when softcap > 0, then (dist_amp, dist_rate, both [heads], not with pooled
+ * blocks) a distance bias dist_amp[h] * ln(1 + dist_rate[h] * (i - j)) is taken off.  q_temp [heads] multiplies every query head after its
+ * norm.  One softmax over everything visible; sink != 0 adds
  * 1 to its denominator (a key of score 0 without a value).  Query head h reads key / value head h / (heads / kv_heads).
  * norm_mode: RMS norm of q and k before rotation — LP_QKNORM_NONE, LP_QKNORM_HEAD (over each head's dim, gains [dim] shared by the
  * heads) or LP_QKNORM_FULL (over the whole projection, gains [heads * dim] and [kv_heads * dim]); both gains NULL: a norm without gains.  q and k are rotated on the first
@@ -719,6 +724,8 @@ typedef struct lp_window_attn_desc {
   int chunk;                                /* > 0: block-local visibility (above) */
   int kv_shared;                            /* != 0: `cache` is another layer's, already written for this step's rows: lp_window_attn_prep
                                                prepares the queries only and qkv holds no keys or values */
+  const float* q_temp;                      /* [heads] or NULL */
+  const float* dist_amp; const float* dist_rate;   /* [heads] each, or both NULL */
 } lp_window_attn_desc;
 /* norm + rotation of the step's rows; keys and values go to the request's pages */
 int lp_window_attn_prep(const lp_window_attn_desc* desc, int R, const int* row_seq, const int* row_pos, void* stream);
@@ -790,6 +797,21 @@ int lp_add_row_f32(float* x, long long ldx, const float* v, int M, int N, void* 
 int lp_token_shift_f32(const float* h, long long ldh, const float* mu, int R, int D, const int* row_seq, const int* row_pos,
                        const int* seq_row0, const int* seq_slot, float* state, long long slot_stride, void* out, long long ldo,
                        int out_fp32, void* stream);
+
+/* short causal convolution added to its input: out_t = h_t + sum_k w[k] * h_(t - taps + 1 + k) per channel, w fp32 [taps][D].  The taps - 1
+ * inputs before a request's first row of the step are the request's slot of `state` (taps - 1 rows of D, oldest first; zeros before
+ * position 0), which afterwards holds the request's last taps - 1 inputs.  The chunk tables are those of lp_retention_prefill, longest_chunk
+ * the most rows one of them has.  1 <= taps <= lp_causal_conv_max_taps() (with one tap there is no state).  Not in place. */
+int lp_causal_conv_max_taps(void);
+int lp_causal_conv_f32(const float* h, long long ldh, const float* w, int taps, int D, int n_chunks, const int* chunk_seq,
+                       const int* chunk_row0, const int* chunk_len, int longest_chunk, const int* row_pos, const int* seq_row0,
+                       const int* seq_slot, float* state, long long slot_stride, void* out, long long ldo, int out_fp32, void* stream);
+/* the norm after the residual sum, in place: x <- z / sqrt(mean(z^2) + eps) * gain[c] with z = alpha x + y.  `out` (NULL: none) receives
+ * the next sublayer's operand: the new x, or — with conv_w [taps][D], one-token steps only (row m is request m at row_pos[m], its slot
+ * row_slot[m]) — the new x with that sublayer's causal convolution added, the slot moving on by one row as in lp_causal_conv_f32. */
+int lp_post_norm_f32(float* x, long long ldx, const float* y, long long ldy, float alpha, int M, int D, const float* gain, float eps,
+                     void* out, long long ldo, int out_fp32, const float* conv_w, int taps, const int* row_pos, const int* row_slot,
+                     float* state, long long slot_stride, void* stream);
 
 /* y <- y + alpha * x over fp32 [M, N] (the residual update after a product that ran on the tensor cores) */
 int lp_axpy_f32(float* y, long long ldy, const float* x, long long ldx, float alpha, int M, int N, void* stream);

@@ -77,8 +77,8 @@ class ProfileRecord(C.Structure):
 
 _P = C.POINTER
 
-EPI_NONE, EPI_XIELU, EPI_SILU_GATE, EPI_RELU2, EPI_CLAMP_GLU = 0, 1, 2, 3, 4
-GATED_EPIS = (EPI_SILU_GATE, EPI_CLAMP_GLU)      # W = [gate rows; up rows], half as many output columns
+EPI_NONE, EPI_XIELU, EPI_SILU_GATE, EPI_RELU2, EPI_CLAMP_GLU, EPI_GELU_GATE = 0, 1, 2, 3, 4, 5
+GATED_EPIS = (EPI_SILU_GATE, EPI_CLAMP_GLU, EPI_GELU_GATE)      # W = [gate rows; up rows], half as many output columns
 RET_FINISH_GATED_NORM, RET_FINISH_RAW = 0, 1
 QKNORM_NONE, QKNORM_HEAD, QKNORM_FULL = 0, 1, 2
 ROT_HALF, ROT_INTERLEAVED = 0, 1
@@ -89,7 +89,8 @@ class LinearDesc(C.Structure):
     """lp_linear_desc (include/leopard_b200.h)."""
     _fields_ = [("A", _vp), ("lda", _ll), ("a_batch", _ll), ("a_fp32", _i), ("W", _vp), ("ldw", _ll), ("w_batch", _ll), ("C", _vp),
                 ("ldc", _ll), ("c_batch", _ll), ("c_fp32", _i), ("M", _i), ("N", _i), ("K", _i), ("batch", _i), ("epi", _i),
-                ("epi_a", _f), ("epi_b", _f), ("c_accum", _i), ("c_scale", _f), ("bias", _vp), ("row_scale", _vp), ("gate", _vp), ("ldg", _ll)]
+                ("epi_a", _f), ("epi_b", _f), ("c_accum", _i), ("c_scale", _f), ("bias", _vp), ("row_scale", _vp), ("gate", _vp), ("ldg", _ll),
+                ("gate_batch", _ll)]
 
 
 class WindowAttnDesc(C.Structure):
@@ -99,7 +100,8 @@ class WindowAttnDesc(C.Structure):
                 ("rot_layout", _i), ("rot_mscale", _f), ("v_inv_freq", _vp), ("v_rot_dims", _i), ("v_rot_layout", _i), ("cache", _vp),
                 ("page_size", _i), ("page_table", _vp), ("max_pages", _i), ("pooled", _vp), ("pooled_table", _vp),
                 ("max_pooled_pages", _i), ("pool", _i), ("window", _i), ("keep_first", _i), ("scale", _f), ("softcap", _f), ("sink", _i),
-                ("q_bias", _vp), ("k_bias", _vp), ("v_bias", _vp), ("v_norm", _i), ("talk", _vp), ("g_off", _i), ("chunk", _i), ("kv_shared", _i)]
+                ("q_bias", _vp), ("k_bias", _vp), ("v_bias", _vp), ("v_norm", _i), ("talk", _vp), ("g_off", _i), ("chunk", _i), ("kv_shared", _i),
+                ("q_temp", _vp), ("dist_amp", _vp), ("dist_rate", _vp)]
 
 
 class MinGRUDesc(C.Structure):
@@ -233,6 +235,9 @@ _SIGS = {
     "lp_add_positions_f32": (_i, [_vp, _ll, _i, _i, _vp, _vp, _vp]),
     "lp_add_row_f32": (_i, [_vp, _ll, _vp, _i, _i, _vp]),
     "lp_token_shift_f32": (_i, [_vp, _ll, _vp, _i, _i, _vp, _vp, _vp, _vp, _vp, _ll, _vp, _ll, _i, _vp]),
+    "lp_causal_conv_max_taps": (_i, []),
+    "lp_causal_conv_f32": (_i, [_vp, _ll, _vp, _i, _i, _i, _vp, _vp, _vp, _i, _vp, _vp, _vp, _vp, _ll, _vp, _ll, _i, _vp]),
+    "lp_post_norm_f32": (_i, [_vp, _ll, _vp, _ll, _f, _i, _i, _vp, _f, _vp, _ll, _i, _vp, _i, _vp, _vp, _vp, _ll, _vp]),
     "lp_moe_route_softmax": (_i, [_vp, _ll, _i, _i, _i, _vp, _ll, _i, _vp, _i, _vp, _vp, _vp]),
     "lp_mingru_workspace_bytes": (_sz, [_i, _i]),
     "lp_mingru_prefill": (_i, [C.POINTER(MinGRUDesc), _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _sz, _vp]),
@@ -303,7 +308,8 @@ STREAM32_SYMBOLS = ("lp_last_error", "lp_abi_version", "lp_launch_count", "lp_li
                     "lp_mingru_workspace_bytes",
                     "lp_mingru_prefill", "lp_mingru_decode", "lp_window_attn_talk", "lp_window_attn_talk_tiles", "lp_mlstm_workspace_bytes", "lp_mlstm",
                     "lp_add_positions_f32", "lp_add_row_f32", "lp_token_shift_f32", "lp_moe_route_softmax", "lp_glu_scaled_f32", "lp_dyt_f32",
-                    "lp_rmsnorm_gated_f32", "lp_gated_axpy_f32", "lp_depth_average_f32", "lp_moe_route_sigmoid", "lp_moe_sorted_weights")
+                    "lp_rmsnorm_gated_f32", "lp_gated_axpy_f32", "lp_depth_average_f32", "lp_moe_route_sigmoid", "lp_moe_sorted_weights",
+                    "lp_causal_conv_max_taps", "lp_causal_conv_f32", "lp_post_norm_f32")
 STREAM32_OPTIONAL = ("lp_gemm_bf16",)      # present in the native libraries, absent from the CPU-emulated build
 _stream32 = None
 

@@ -2,8 +2,8 @@
 //
 //   lp_linear          C[M,N] = epi(A[M,K] · W[N,K]^T): A fp32 or bf16, W bf16 (nn.Linear layout), C fp32 or bf16, accumulation in
 //                      fp32 FMAs in index order of K (no tensor-core rounding: with fp32 A this is a true 32-bit product, the bf16
-//                      weight is exact in fp32).  Epilogues: none, xIELU, squared relu, gated SiLU and the clamped gated unit (W =
-//                      [gate rows; up rows], C has N/2 columns).  Before the epilogue every accumulator may be multiplied by a
+//                      weight is exact in fp32).  Epilogues: none, xIELU, squared relu, and the gated units silu, gelu (tanh form)
+//                      and the clamped one (W = [gate rows; up rows], C has N/2 columns).  Before the epilogue every accumulator may be multiplied by a
 //                      number per output row (row_scale: a router weight that multiplies an expert's INPUT is the same as one
 //                      that multiplies its first products) and take a bias per weight row.  With c_accum the result is scaled
 //                      and ADDED to C (the residual update of a pre-norm layer); with `gate` it is first multiplied by
@@ -39,7 +39,7 @@ struct LinArgs {
   int a_div;
   const float* bias;      // [N] added to the accumulators before the epilogue, or NULL
   const float* row_scale; // [rows of C] multiplies the accumulators before the bias, or NULL
-  const float* gate; long long ldg;   // [rows of C, N'] pre-activations: the result is multiplied by sigmoid(gate), or NULL
+  const float* gate; long long ldg, gate_batch;   // [rows of C, N'] pre-activations: the result is multiplied by sigmoid(gate), or NULL
 };
 
 __device__ __forceinline__ float lin_load(const float* p) { return *p; }
@@ -69,13 +69,20 @@ __device__ __forceinline__ float lin_epi(int epi, float v, float e0, float e1) {
   return epi == LP_EPI_XIELU ? xielu_f(v, e0, e1) : v;
 }
 
-// the two gated units: silu(g) * u, and g' sigmoid(e1 g') (u' + 1) with g' = min(g, e0), u' = clamp(u, -e0, e0)
+// tanh-form gelu: 1/2 (1 + tanh t) is sigmoid(2 t), so one exponential serves
+__device__ __forceinline__ float gelu_tanh32_f(float z) {
+  const float t = 0.7978845608028654f * fmaf(0.044715f * z * z, z, z);      // sqrt(2 / pi) (z + 0.044715 z^3)
+  return z / (1.0f + expf(-2.0f * t));
+}
+
+// the gated units: silu(g) * u, gelu(g) * u, and g' sigmoid(e1 g') (u' + 1) with g' = min(g, e0), u' = clamp(u, -e0, e0)
 __device__ __forceinline__ float lin_gate(int epi, float g, float u, float e0, float e1) {
   if (epi == LP_EPI_CLAMP_GLU) {
     g = fminf(g, e0);
     u = fminf(fmaxf(u, -e0), e0);
     return g / (1.0f + expf(-e1 * g)) * (u + 1.0f);
   }
+  if (epi == LP_EPI_GELU_GATE) return gelu_tanh32_f(g) * u;
   return silu32_f(g) * u;
 }
 
@@ -86,16 +93,16 @@ __global__ void __launch_bounds__(LIN_THREADS) linear_tile_kernel(LinArgs a) {
   __shared__ float As[LIN_BK][LIN_BM + 4];
   __shared__ float Ws[GATED ? 2 : 1][LIN_BK][LIN_BN + 4];
   const int tid = threadIdx.x;
-  const int tile_m = blockIdx.y, tile_n = blockIdx.x, z = blockIdx.z;
+  const int tile_m = blockIdx.y, tile_n = blockIdx.x, z_id = blockIdx.z;
   int group = 0;
   if (a.tile_group != nullptr) {
     group = a.tile_group[tile_m];
     if (group < 0) return;
   }
   const int n_out = GATED ? a.N / 2 : a.N;
-  const AT* A = reinterpret_cast<const AT*>(a.A) + (long long)z * a.a_batch;
-  const bf16* W = a.W + (long long)(z + group) * a.w_batch;   // grouped launches have one batch: z = 0
-  CT* C = reinterpret_cast<CT*>(a.C) + (long long)z * a.c_batch;
+  const AT* A = reinterpret_cast<const AT*>(a.A) + (long long)z_id * a.a_batch;
+  const bf16* W = a.W + (long long)(z_id + group) * a.w_batch;   // grouped launches have one batch: z_id = 0
+  CT* C = reinterpret_cast<CT*>(a.C) + (long long)z_id * a.c_batch;
   const int m0 = tile_m * LIN_BM, n0 = tile_n * LIN_BN;
   // loader mapping: 256 threads x 4 elements = 64 rows x 16 k
   const int lr = tid >> 2, lk = (tid & 3) * 4;
@@ -157,7 +164,7 @@ __global__ void __launch_bounds__(LIN_THREADS) linear_tile_kernel(LinArgs a) {
         if (GATED) z2 += a.bias[n + n_out];
       }
       float v = GATED ? lin_gate(a.epi, z, z2, a.e0, a.e1) : lin_epi(a.epi, z, a.e0, a.e1);
-      if (a.gate != nullptr) v /= 1.0f + expf(-a.gate[(long long)m * a.ldg + n]);
+      if (a.gate != nullptr) v /= 1.0f + expf(-a.gate[(long long)z_id * a.gate_batch + (long long)m * a.ldg + n]);
       if (a.c_accum) v = fmaf(a.c_scale, v, lin_load(C + (long long)m * a.ldc + n));
       lin_store(C + (long long)m * a.ldc + n, v);
     }
@@ -257,7 +264,7 @@ __global__ void __launch_bounds__(ROWS_WARPS * 32) linear_rows_kernel(LinArgs a)
           if (GATED) s2 += a.bias[n + n_out];
         }
         float v = GATED ? lin_gate(a.epi, s, s2, a.e0, a.e1) : lin_epi(a.epi, s, a.e0, a.e1);
-        if (a.gate != nullptr) v /= 1.0f + expf(-a.gate[(long long)(pairs ? z : m) * a.ldg + n]);
+        if (a.gate != nullptr) v /= 1.0f + expf(-a.gate[(pairs ? 0 : (long long)z * a.gate_batch) + (long long)(pairs ? z : m) * a.ldg + n]);
         if (a.c_accum) v = fmaf(a.c_scale, v, lin_load(C + (long long)m * a.ldc + n));
         lin_store(C + (long long)m * a.ldc + n, v);
       }
@@ -280,8 +287,10 @@ static int launch_linear(const LinArgs& a, int batch, int m_tiles, bool allow_ro
   return 0;
 }
 
+static bool gated_epi(int epi) { return epi == LP_EPI_SILU_GATE || epi == LP_EPI_CLAMP_GLU || epi == LP_EPI_GELU_GATE; }
+
 static int dispatch_linear(const LinArgs& a, int a_fp32, int c_fp32, int batch, int m_tiles, bool allow_rows, cudaStream_t stream) {
-  const bool gated = a.epi == LP_EPI_SILU_GATE || a.epi == LP_EPI_CLAMP_GLU;
+  const bool gated = gated_epi(a.epi);
   if (a_fp32) {
     if (c_fp32) return gated ? launch_linear<float, float, true>(a, batch, m_tiles, allow_rows, stream)
                              : launch_linear<float, float, false>(a, batch, m_tiles, allow_rows, stream);
@@ -303,8 +312,8 @@ extern "C" int lp_linear(const lp_linear_desc* d, void* stream_) {
   LP_REQUIRE(d != nullptr && d->A != nullptr && d->W != nullptr && d->C != nullptr, "lp_linear: null operand");
   LP_REQUIRE(d->M >= 0 && d->N > 0 && d->K > 0 && d->batch >= 1, "lp_linear: bad problem M=%d N=%d K=%d batch=%d", d->M, d->N, d->K,
              d->batch);
-  LP_REQUIRE(d->epi >= LP_EPI_NONE && d->epi <= LP_EPI_CLAMP_GLU, "lp_linear: bad epilogue %d", d->epi);
-  LP_REQUIRE((d->epi != LP_EPI_SILU_GATE && d->epi != LP_EPI_CLAMP_GLU) || d->N % 2 == 0, "lp_linear: the gated epilogue needs an even N (gate rows, then up rows)");
+  LP_REQUIRE(d->epi >= LP_EPI_NONE && d->epi <= LP_EPI_GELU_GATE, "lp_linear: bad epilogue %d", d->epi);
+  LP_REQUIRE(!gated_epi(d->epi) || d->N % 2 == 0, "lp_linear: the gated epilogue needs an even N (gate rows, then up rows)");
   if (d->M == 0) return 0;
   LinArgs a;
   a.A = d->A; a.lda = d->lda; a.a_batch = d->a_batch;
@@ -313,7 +322,7 @@ extern "C" int lp_linear(const lp_linear_desc* d, void* stream_) {
   a.M = d->M; a.N = d->N; a.K = d->K;
   a.epi = d->epi; a.e0 = d->epi_a; a.e1 = d->epi_b; a.c_accum = d->c_accum; a.c_scale = d->c_scale;
   a.a_rows = nullptr; a.tile_group = nullptr; a.z_group = nullptr; a.a_div = 1;
-  a.bias = d->bias; a.row_scale = d->row_scale; a.gate = d->gate; a.ldg = d->ldg;
+  a.bias = d->bias; a.row_scale = d->row_scale; a.gate = d->gate; a.ldg = d->ldg; a.gate_batch = d->gate_batch;
   LP_REQUIRE(d->batch == 1 || (d->bias == nullptr && d->row_scale == nullptr), "lp_linear: bias and row scale are for one problem");
   return dispatch_linear(a, d->a_fp32, d->c_fp32, d->batch, (d->M + LIN_BM - 1) / LIN_BM, true, stream);
 }
@@ -325,8 +334,8 @@ extern "C" int lp_linear_pairs(const lp_linear_desc* d, const int* pair_group, i
   LP_REQUIRE(d != nullptr && d->A != nullptr && d->W != nullptr && d->C != nullptr && pair_group != nullptr, "lp_linear_pairs: null operand");
   LP_REQUIRE(d->N > 0 && d->K > 0 && a_div >= 1 && n_pairs >= 0 && n_pairs <= 65535, "lp_linear_pairs: bad problem N=%d K=%d pairs=%d", d->N,
              d->K, n_pairs);
-  LP_REQUIRE(d->epi >= LP_EPI_NONE && d->epi <= LP_EPI_CLAMP_GLU, "lp_linear_pairs: bad epilogue %d", d->epi);
-  LP_REQUIRE((d->epi != LP_EPI_SILU_GATE && d->epi != LP_EPI_CLAMP_GLU) || d->N % 2 == 0, "lp_linear_pairs: the gated epilogue needs an even N");
+  LP_REQUIRE(d->epi >= LP_EPI_NONE && d->epi <= LP_EPI_GELU_GATE, "lp_linear_pairs: bad epilogue %d", d->epi);
+  LP_REQUIRE(!gated_epi(d->epi) || d->N % 2 == 0, "lp_linear_pairs: the gated epilogue needs an even N");
   if (n_pairs == 0) return 0;
   LinArgs a;
   a.A = d->A; a.lda = d->lda; a.a_batch = 0;
@@ -335,7 +344,7 @@ extern "C" int lp_linear_pairs(const lp_linear_desc* d, const int* pair_group, i
   a.M = 1; a.N = d->N; a.K = d->K;
   a.epi = d->epi; a.e0 = d->epi_a; a.e1 = d->epi_b; a.c_accum = d->c_accum; a.c_scale = d->c_scale;
   a.a_rows = nullptr; a.tile_group = nullptr; a.z_group = pair_group; a.a_div = a_div;
-  a.bias = d->bias; a.row_scale = d->row_scale; a.gate = d->gate; a.ldg = d->ldg;
+  a.bias = d->bias; a.row_scale = d->row_scale; a.gate = d->gate; a.ldg = d->ldg; a.gate_batch = d->gate_batch;
   return dispatch_linear(a, d->a_fp32, d->c_fp32, n_pairs, 1, true, stream);
 }
 
@@ -344,8 +353,8 @@ extern "C" int lp_linear_grouped(const lp_linear_desc* d, const int* tile_group,
   LP_REQUIRE(d != nullptr && d->A != nullptr && d->W != nullptr && d->C != nullptr && tile_group != nullptr,
              "lp_linear_grouped: null operand");
   LP_REQUIRE(d->N > 0 && d->K > 0 && n_tiles >= 0, "lp_linear_grouped: bad problem N=%d K=%d tiles=%d", d->N, d->K, n_tiles);
-  LP_REQUIRE(d->epi >= LP_EPI_NONE && d->epi <= LP_EPI_CLAMP_GLU, "lp_linear_grouped: bad epilogue %d", d->epi);
-  LP_REQUIRE((d->epi != LP_EPI_SILU_GATE && d->epi != LP_EPI_CLAMP_GLU) || d->N % 2 == 0, "lp_linear_grouped: the gated epilogue needs an even N");
+  LP_REQUIRE(d->epi >= LP_EPI_NONE && d->epi <= LP_EPI_GELU_GATE, "lp_linear_grouped: bad epilogue %d", d->epi);
+  LP_REQUIRE(!gated_epi(d->epi) || d->N % 2 == 0, "lp_linear_grouped: the gated epilogue needs an even N");
   if (n_tiles == 0) return 0;
   LinArgs a;
   a.A = d->A; a.lda = d->lda; a.a_batch = 0;
@@ -354,7 +363,7 @@ extern "C" int lp_linear_grouped(const lp_linear_desc* d, const int* tile_group,
   a.M = n_tiles * LIN_BM; a.N = d->N; a.K = d->K;
   a.epi = d->epi; a.e0 = d->epi_a; a.e1 = d->epi_b; a.c_accum = d->c_accum; a.c_scale = d->c_scale;
   a.a_rows = a_rows; a.tile_group = tile_group; a.z_group = nullptr; a.a_div = 1;
-  a.bias = d->bias; a.row_scale = d->row_scale; a.gate = d->gate; a.ldg = d->ldg;
+  a.bias = d->bias; a.row_scale = d->row_scale; a.gate = d->gate; a.ldg = d->ldg; a.gate_batch = d->gate_batch;
   return dispatch_linear(a, d->a_fp32, d->c_fp32, 1, n_tiles, false, stream);
 }
 

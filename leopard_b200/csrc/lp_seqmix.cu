@@ -18,9 +18,10 @@
 //                        The kernels work on the cache directly (absorbed form): score = (W_uk^T q_unrot) . c + q_rot . k_rot, output =
 //                        W_uv (sum_j p_j c_j); the two per-head products run as batched lp_linear calls around lp_latent_attend.
 //                        Sliding window: key j is visible to query i when 0 <= i - j < window (window <= 0: all earlier keys).
-//                        Cache: pages of `page_size` rows [c | k_rot] fp32, one page table row per request.
+//                        Cache: pages of `page_size` rows [c | k_rot] fp32, one page table row per request.  Layers may share one cache:
+//                        a layer without latents of its own (dkv NULL) reads the rows another layer wrote earlier in the step.
 //       lp_latent_prep   RMS-norms the latent (vector gain), rotates the shared key part and writes both to the request's pages;
-//                        rotates the query's rotated part in place.
+//                        rotates the query's rotated part in place (without latents of its own: only that).
 //       lp_latent_attend one CTA per (row, head), its warps split the visible keys: online softmax in fp32, merged at the end.
 #include "lp_host.h"
 #include "../../include/leopard_b200.h"
@@ -410,18 +411,20 @@ latent_prep_kernel(LatArgs a, int R, const int* __restrict__ row_seq, const int*
   const int r = blockIdx.x, tid = threadIdx.x;
   if (r >= R) return;
   const int pos = row_pos[r];
-  const float* src = a.dkv + (long long)r * a.lddkv;
-  float ss = 0.f;
-  for (int c = tid; c < a.kv_rank; c += blockDim.x) ss = fmaf(src[c], src[c], ss);
+  if (a.dkv != nullptr) {      // the layer brings latents of its own
+    const float* src = a.dkv + (long long)r * a.lddkv;
+    float ss = 0.f;
+    for (int c = tid; c < a.kv_rank; c += blockDim.x) ss = fmaf(src[c], src[c], ss);
 #pragma unroll
-  for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-  if ((tid & 31) == 0) red[tid >> 5] = ss;
-  __syncthreads();
-  const float inv = 1.0f / sqrtf((red[0] + red[1] + red[2] + red[3]) / (float)a.kv_rank + a.eps);
-  float* dst = lat_cache_row(a, row_seq[r], pos);
-  for (int c = tid; c < a.kv_rank; c += blockDim.x) dst[c] = src[c] * inv * a.c_gain[c];
-  for (int d = tid; d < a.rot_dim; d += blockDim.x)
-    dst[a.kv_rank + d] = rot_elem(src + a.kv_rank, d, a.rot_dims, a.rot_layout, a.inv_freq, a.rot_mscale, pos);
+    for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    if ((tid & 31) == 0) red[tid >> 5] = ss;
+    __syncthreads();
+    const float inv = 1.0f / sqrtf((red[0] + red[1] + red[2] + red[3]) / (float)a.kv_rank + a.eps);
+    float* dst = lat_cache_row(a, row_seq[r], pos);
+    for (int c = tid; c < a.kv_rank; c += blockDim.x) dst[c] = src[c] * inv * a.c_gain[c];
+    for (int d = tid; d < a.rot_dim; d += blockDim.x)
+      dst[a.kv_rank + d] = rot_elem(src + a.kv_rank, d, a.rot_dims, a.rot_layout, a.inv_freq, a.rot_mscale, pos);
+  }
   // the rotated part of every head's query, in place: one thread per pair reads both members, then writes both
   float* q = a.q + (long long)r * a.ldq;
   const int per = a.dim + a.rot_dim, half = a.rot_dims >> 1;
@@ -709,7 +712,7 @@ extern "C" int lp_latent_prep(const lp_latent_desc* d, int R, const int* row_seq
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
   LatArgs a;
   if (int rc = fill_lat(a, d)) return rc;
-  LP_REQUIRE(d->dkv != nullptr && d->c_gain != nullptr && row_seq != nullptr && row_pos != nullptr, "lp_latent_prep: null operand");
+  LP_REQUIRE((d->dkv == nullptr || d->c_gain != nullptr) && row_seq != nullptr && row_pos != nullptr, "lp_latent_prep: null operand");
   if (R <= 0) return 0;
   latent_prep_kernel<<<R, 128, 0, stream>>>(a, R, row_seq, row_pos);
   note_launch();

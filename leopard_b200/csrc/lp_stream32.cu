@@ -4,7 +4,7 @@
 //   lp_rmsnorm_f32      y = x / sqrt(mean(x^2) + eps) * g over fp32 rows, eps inside the root; g is one number (gain_scalar), a vector
 //                       (gain_vec) or both.  The result is written as fp32 or bf16 (the operand of the next matrix product), or — with
 //                       `accum` — added to another fp32 matrix: the sandwich-norm residual update x <- x + norm(sublayer(x)) in one pass.
-//   lp_glu_f32          elementwise epilogues for matrix products that ran elsewhere: xIELU, squared relu, silu(gate) * up.
+//   lp_glu_f32          elementwise epilogues for matrix products that ran elsewhere: xIELU, squared relu, silu(gate) * up, gelu(gate) * up.
 //   lp_axpy_f32         y <- y + alpha x, the residual update after such a product.
 //   lp_add_positions_f32  x[r, 2i] += sin(p f_i), x[r, 2i + 1] += cos(p f_i) with p the row's position: absolute sinusoidal positions
 //                       added to the stream (fp32 angles with the product's rounding error carried along, accurate sincosf).
@@ -12,6 +12,11 @@
 //   lp_token_shift_f32  y_t = h_t + (h_(t-1) - h_t) * mu per channel, with h the rows as they came in; the row before a request's
 //                       first row of this step comes from the request's slot (zeros at position 0), and the slot then takes the
 //                       request's last row.
+//   lp_causal_conv_f32  out_t = h_t + sum_j w_j h_(t - K + 1 + j) per channel: a short causal convolution added to its input; the K - 1
+//                       inputs before a request's first row of this step come from the request's slot (zeros before position 0), and
+//                       the slot then takes the request's last K - 1 inputs.
+//   lp_post_norm_f32    x <- norm(alpha x + y) * gain, the norm after the residual sum, in place; the same pass writes the next sublayer's
+//                       operand: the new x, for one-token steps with the next sublayer's causal convolution applied on the way.
 //   lp_dyt_f32          Dynamic Tanh: tanh(alpha x) * gain + shift per element, no statistics; one pass can serve the two sublayers of a
 //                       parallel layer (two parameter sets, two outputs).
 //   lp_rmsnorm_gated_f32  the RMS norm with a vector gain, multiplied by sigmoid(gate) per element (norm over a mixer's concatenated
@@ -70,7 +75,8 @@ template <> __device__ __forceinline__ float ld32<bf16>(const bf16* p) { return 
 __device__ __forceinline__ void st32(float* p, float v) { *p = v; }
 __device__ __forceinline__ void st32(bf16* p, float v) { *p = __float2bfloat16(v); }
 
-// mode LP_EPI_XIELU: out[m, n] = xielu(in[m, n]); LP_EPI_SILU_GATE: out[m, n] = silu(in[m, n]) * in[m, n + N]; LP_EPI_CLAMP_GLU: the
+// mode LP_EPI_XIELU: out[m, n] = xielu(in[m, n]); LP_EPI_SILU_GATE, LP_EPI_GELU_GATE:
+// out[m, n] = silu | gelu (in[m, n]) * in[m, n + N]; LP_EPI_CLAMP_GLU: the
 // clamped gated unit of lp_linear on (in[m, n], in[m, n + N]) with limit a and slope b.  row_scale multiplies what is read.
 template <typename IT, typename OT>
 __global__ void glu_kernel(const IT* __restrict__ in, long long ldi, OT* __restrict__ out, long long ldo, int M, int N, int mode, float a,
@@ -82,6 +88,10 @@ __global__ void glu_kernel(const IT* __restrict__ in, long long ldi, OT* __restr
   const float z = ld32<IT>(in + (long long)m * ldi + n) * rs;
   float v;
   if (mode == LP_EPI_SILU_GATE) v = z / (1.0f + expf(-z)) * (ld32<IT>(in + (long long)m * ldi + n + N) * rs);
+  else if (mode == LP_EPI_GELU_GATE) {      // tanh form: 1/2 (1 + tanh t) = sigmoid(2 t) with t = sqrt(2 / pi) (z + 0.044715 z^3)
+    const float t = 0.7978845608028654f * fmaf(0.044715f * z * z, z, z);
+    v = z / (1.0f + expf(-2.0f * t)) * (ld32<IT>(in + (long long)m * ldi + n + N) * rs);
+  }
   else if (mode == LP_EPI_CLAMP_GLU) {
     const float g = fminf(z, a), u = fminf(fmaxf(ld32<IT>(in + (long long)m * ldi + n + N) * rs, -a), a);
     v = g / (1.0f + expf(-b * g)) * (u + 1.0f);
@@ -285,9 +295,268 @@ __global__ void token_shift_kernel(const float* __restrict__ h, long long ldh, c
   st32(out + (long long)r * ldo + c, fmaf(prev - cur, mu[c], cur));
 }
 
+// Short causal convolution added to its input.  A thread owns V channels of one TILE of consecutive rows of a request and walks the
+// rows with the K - 1 inputs before them in registers.  Tiles (and full chunks) are at least K - 1 rows long, so only the thread of a
+// request's FIRST tile reaches back past the rows of this step into the request's slot: it reads the carried inputs and then stores
+// the request's last K - 1 inputs there, and no other thread of the launch touches them.  The slot holds K - 1 rows of D, oldest
+// first, zeros for positions before the request's start.
+template <typename OT, int V, int K>
+__global__ void causal_conv_kernel(const float* __restrict__ h, long long ldh, const float* __restrict__ w, int D, const int* __restrict__ chunk_seq,
+                                   const int* __restrict__ chunk_row0, const int* __restrict__ chunk_len, int subs, int tile,
+                                   const int* __restrict__ row_pos, const int* __restrict__ seq_row0, const int* __restrict__ seq_slot,
+                                   float* __restrict__ state, long long slot_stride, OT* __restrict__ out, long long ldo) {
+  const int ck = blockIdx.x / subs, sub = blockIdx.x % subs;
+  const int c = (blockIdx.y * blockDim.x + threadIdx.x) * V;
+  if (sub * tile >= chunk_len[ck] || c >= D) return;
+  const int s = chunk_seq[ck], first = seq_row0[s], end = seq_row0[s + 1];
+  const int r0 = chunk_row0[ck] + sub * tile, rows = min(tile, chunk_len[ck] - sub * tile);
+  const bool started = row_pos[first] > 0;      // earlier steps left inputs in the slot
+  float* slot = state + (long long)seq_slot[s] * slot_stride + c;
+  f32vec<V> wv[K], win[K];      // win[k]: the input K - 1 - k rows before the current one; win[K - 1] the current one
+#pragma unroll
+  for (int k = 0; k < K; ++k) {
+    wv[k] = ldv<V>(w + (long long)k * D + c);
+#pragma unroll
+    for (int i = 0; i < V; ++i) win[k].v[i] = 0.f;
+  }
+#pragma unroll
+  for (int k = 0; k < K - 1; ++k) {
+    const int r = r0 - (K - 1) + k;
+    if (r >= first) win[k] = ldv<V>(h + (long long)r * ldh + c);
+    else if (started) win[k] = ldv<V>(slot + (long long)(K - 1 + r - first) * D);
+  }
+  if (K > 1 && r0 == first) {
+    f32vec<V> zero;
+#pragma unroll
+    for (int i = 0; i < V; ++i) zero.v[i] = 0.f;
+    for (int k = 0; k < K - 1; ++k) {      // row end - (K - 1) + k; a carried one moves towards the slot's start, so in place is safe
+      const int r = end - (K - 1) + k;
+      stv<V>(slot + (long long)k * D, r >= first ? ldv<V>(h + (long long)r * ldh + c) : started ? ldv<V>(slot + (long long)(K - 1 + r - first) * D) : zero);
+    }
+  }
+  for (int t = 0; t < rows; ++t) {
+    const long long r = r0 + t;
+    win[K - 1] = ldv<V>(h + r * ldh + c);
+    f32vec<V> y = win[K - 1];
+#pragma unroll
+    for (int k = 0; k < K; ++k)
+#pragma unroll
+      for (int i = 0; i < V; ++i) y.v[i] = fmaf(wv[k].v[i], win[k].v[i], y.v[i]);
+    stv<V>(out + r * ldo + c, y);
+#pragma unroll
+    for (int k = 0; k < K - 1; ++k) win[k] = win[k + 1];
+  }
+}
+
+// More taps than the register window holds: one channel per thread, every input read again for every tap.  The same ownership of the
+// slot, which the thread of a request's first tile rewrites after its last row.
+template <typename OT>
+__global__ void causal_conv_long_kernel(const float* __restrict__ h, long long ldh, const float* __restrict__ w, int K, int D,
+                                        const int* __restrict__ chunk_seq, const int* __restrict__ chunk_row0, const int* __restrict__ chunk_len,
+                                        const int* __restrict__ row_pos, const int* __restrict__ seq_row0, const int* __restrict__ seq_slot,
+                                        float* state, long long slot_stride, OT* __restrict__ out, long long ldo) {
+  const int ck = blockIdx.x, c = blockIdx.y * blockDim.x + threadIdx.x;
+  if (c >= D) return;
+  const int s = chunk_seq[ck], first = seq_row0[s], end = seq_row0[s + 1], r0 = chunk_row0[ck];
+  const bool started = row_pos[first] > 0;
+  float* slot = state + (long long)seq_slot[s] * slot_stride + c;
+  auto input = [&](int r) {
+    if (r >= first) return h[(long long)r * ldh + c];
+    return started ? slot[(long long)(K - 1 + r - first) * D] : 0.f;
+  };
+  for (int r = r0; r < r0 + chunk_len[ck]; ++r) {
+    float y = h[(long long)r * ldh + c];
+    for (int k = 0; k < K; ++k) y = fmaf(w[(long long)k * D + c], input(r - (K - 1) + k), y);
+    st32(out + (long long)r * ldo + c, y);
+  }
+  if (r0 == first)
+    for (int k = 0; k < K - 1; ++k) slot[(long long)k * D] = input(end - (K - 1) + k);      // reads ahead of what it writes
+}
+
+// a full chunk is as long as the inputs a row looks back at, so no chunk but a request's first needs the slot
+constexpr int CONV_WINDOW_TAPS = 8, CONV_MAX_TAPS = LP_RETENTION_CHUNK + 1, CONV_TILE = 16, CONV_THREADS = 128;
+
+struct ConvLaunch {
+  const float* h; long long ldh; const float* w; int D;
+  int n_chunks; const int *chunk_seq, *chunk_row0, *chunk_len; int longest;
+  const int *row_pos, *seq_row0, *seq_slot;
+  float* state; long long slot_stride;
+  void* out; long long ldo;
+};
+
+template <typename OT, int V, int K>
+static void launch_conv(const ConvLaunch& a, cudaStream_t stream) {
+  const int subs = (a.longest + CONV_TILE - 1) / CONV_TILE;
+  const dim3 grid(a.n_chunks * subs, (a.D / V + CONV_THREADS - 1) / CONV_THREADS);
+  causal_conv_kernel<OT, V, K><<<grid, CONV_THREADS, 0, stream>>>(a.h, a.ldh, a.w, a.D, a.chunk_seq, a.chunk_row0, a.chunk_len, subs, CONV_TILE,
+                                                                 a.row_pos, a.seq_row0, a.seq_slot, a.state, a.slot_stride,
+                                                                 reinterpret_cast<OT*>(a.out), a.ldo);
+}
+
+template <typename OT, int V>
+static void launch_conv_taps(const ConvLaunch& a, int taps, cudaStream_t stream) {
+  switch (taps) {
+    case 1: launch_conv<OT, V, 1>(a, stream); break;
+    case 2: launch_conv<OT, V, 2>(a, stream); break;
+    case 3: launch_conv<OT, V, 3>(a, stream); break;
+    case 4: launch_conv<OT, V, 4>(a, stream); break;
+    case 5: launch_conv<OT, V, 5>(a, stream); break;
+    case 6: launch_conv<OT, V, 6>(a, stream); break;
+    case 7: launch_conv<OT, V, 7>(a, stream); break;
+    case 8: launch_conv<OT, V, 8>(a, stream); break;
+    default:
+      causal_conv_long_kernel<OT><<<dim3(a.n_chunks, (a.D + CONV_THREADS - 1) / CONV_THREADS), CONV_THREADS, 0, stream>>>(
+          a.h, a.ldh, a.w, taps, a.D, a.chunk_seq, a.chunk_row0, a.chunk_len, a.row_pos, a.seq_row0, a.seq_slot, a.state, a.slot_stride,
+          reinterpret_cast<OT*>(a.out), a.ldo);
+      break;
+  }
+}
+
+// One CTA per row: x <- norm(alpha x + y) * gain, and the next sublayer's operand.  The sums alpha x + y of the first POST_KEEP column groups
+// of a thread stay in registers between the two passes; wider rows park theirs in x.  With conv_w (one-token steps: row m is the only
+// row of request m) the operand is the new x plus the causal convolution over the slot's carried inputs and the new x, and the slot
+// moves on by one row; a thread reads and writes its own columns of the slot only.
+constexpr int POST_THREADS = 256, POST_KEEP = 4;
+template <typename OT, int V>
+__global__ void __launch_bounds__(POST_THREADS)
+post_norm_kernel(float* __restrict__ x, long long ldx, const float* __restrict__ y, long long ldy, float alpha, int D,
+                 const float* __restrict__ gain, float eps, OT* __restrict__ out, long long ldo, const float* __restrict__ conv_w, int taps,
+                 const int* __restrict__ row_pos, const int* __restrict__ row_slot, float* __restrict__ state, long long slot_stride) {
+  __shared__ float red[POST_THREADS / 32];
+  const long long m = blockIdx.x;
+  const int tid = threadIdx.x, step = blockDim.x * V;
+  float* xr = x + m * ldx;
+  const float* yr = y + m * ldy;
+  f32vec<V> keep[POST_KEEP];
+  float ss = 0.f;
+#pragma unroll
+  for (int it = 0; it < POST_KEEP; ++it) {
+    const int c = tid * V + it * step;
+    if (c < D) {
+      const f32vec<V> a = ldv<V>(xr + c), b = ldv<V>(yr + c);
+#pragma unroll
+      for (int i = 0; i < V; ++i) {
+        keep[it].v[i] = fmaf(alpha, a.v[i], b.v[i]);
+        ss = fmaf(keep[it].v[i], keep[it].v[i], ss);
+      }
+    }
+  }
+  for (int c = tid * V + POST_KEEP * step; c < D; c += step) {
+    f32vec<V> a = ldv<V>(xr + c);
+    const f32vec<V> b = ldv<V>(yr + c);
+#pragma unroll
+    for (int i = 0; i < V; ++i) {
+      a.v[i] = fmaf(alpha, a.v[i], b.v[i]);
+      ss = fmaf(a.v[i], a.v[i], ss);
+    }
+    stv<V>(xr + c, a);
+  }
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+  if ((tid & 31) == 0) red[tid >> 5] = ss;
+  __syncthreads();
+  float total = 0.f;
+  for (int k = 0; k < (int)(blockDim.x >> 5); ++k) total += red[k];
+  const float r = 1.0f / sqrtf(total / (float)D + eps);
+  float* slot = nullptr;
+  bool started = false;
+  if (conv_w != nullptr && taps > 1) {
+    slot = state + (long long)row_slot[m] * slot_stride;
+    started = row_pos[m] > 0;
+  }
+  auto finish = [&](int c, f32vec<V> z) {
+    const f32vec<V> g = ldv<V>(gain + c);
+#pragma unroll
+    for (int i = 0; i < V; ++i) z.v[i] = z.v[i] * r * g.v[i];
+    stv<V>(xr + c, z);
+    if (out == nullptr) return;
+    f32vec<V> o = z;
+    if (conv_w != nullptr) {
+      for (int k = 0; k < taps - 1; ++k) {
+        f32vec<V> old;
+#pragma unroll
+        for (int i = 0; i < V; ++i) old.v[i] = 0.f;
+        if (started) old = ldv<V>(slot + (long long)k * D + c);
+        const f32vec<V> wk = ldv<V>(conv_w + (long long)k * D + c);
+#pragma unroll
+        for (int i = 0; i < V; ++i) o.v[i] = fmaf(wk.v[i], old.v[i], o.v[i]);
+        if (k > 0) stv<V>(slot + (long long)(k - 1) * D + c, old);
+      }
+      const f32vec<V> wk = ldv<V>(conv_w + (long long)(taps - 1) * D + c);
+#pragma unroll
+      for (int i = 0; i < V; ++i) o.v[i] = fmaf(wk.v[i], z.v[i], o.v[i]);
+      if (taps > 1) stv<V>(slot + (long long)(taps - 2) * D + c, z);
+    }
+    stv<V>(out + m * ldo + c, o);
+  };
+#pragma unroll
+  for (int it = 0; it < POST_KEEP; ++it) {
+    const int c = tid * V + it * step;
+    if (c < D) finish(c, keep[it]);
+  }
+  for (int c = tid * V + POST_KEEP * step; c < D; c += step) finish(c, ldv<V>(xr + c));
+}
+
 }  // namespace lp
 
 using namespace lp;
+
+extern "C" int lp_causal_conv_max_taps(void) { return CONV_MAX_TAPS; }
+
+extern "C" int lp_causal_conv_f32(const float* h, long long ldh, const float* w, int taps, int D, int n_chunks, const int* chunk_seq,
+                                  const int* chunk_row0, const int* chunk_len, int longest_chunk, const int* row_pos, const int* seq_row0,
+                                  const int* seq_slot, float* state, long long slot_stride, void* out, long long ldo, int out_fp32,
+                                  void* stream_) {
+  cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
+  LP_REQUIRE(h != nullptr && w != nullptr && out != nullptr && chunk_seq != nullptr && chunk_row0 != nullptr && chunk_len != nullptr &&
+                 row_pos != nullptr && seq_row0 != nullptr && seq_slot != nullptr && D > 0 && n_chunks >= 0,
+             "lp_causal_conv_f32: bad arguments");
+  LP_REQUIRE(taps >= 1 && taps <= CONV_MAX_TAPS, "lp_causal_conv_f32: %d taps (1 .. %d are built)", taps, CONV_MAX_TAPS);
+  LP_REQUIRE(taps == 1 || (state != nullptr && slot_stride >= (long long)(taps - 1) * D), "lp_causal_conv_f32: no room for the carried inputs");
+  LP_REQUIRE(longest_chunk >= 1 && longest_chunk <= LP_RETENTION_CHUNK, "lp_causal_conv_f32: longest_chunk=%d", longest_chunk);
+  LP_REQUIRE(h != out, "lp_causal_conv_f32: a row reads its neighbours as they came in, so it cannot run in place");
+  if (n_chunks == 0) return 0;
+  const ConvLaunch a{h, ldh, w, D, n_chunks, chunk_seq, chunk_row0, chunk_len, longest_chunk, row_pos, seq_row0, seq_slot, state, slot_stride, out, ldo};
+  const bool v4 = taps <= CONV_WINDOW_TAPS && vec4_ok(D, {h, w, state, out}, {ldh, ldo, taps > 1 ? slot_stride : 0});
+  if (out_fp32 && v4) launch_conv_taps<float, 4>(a, taps, stream);
+  else if (out_fp32) launch_conv_taps<float, 1>(a, taps, stream);
+  else if (v4) launch_conv_taps<bf16, 4>(a, taps, stream);
+  else launch_conv_taps<bf16, 1>(a, taps, stream);
+  note_launch();
+  LP_CHECK_CUDA(cudaGetLastError());
+  return 0;
+}
+
+extern "C" int lp_post_norm_f32(float* x, long long ldx, const float* y, long long ldy, float alpha, int M, int D, const float* gain, float eps,
+                                void* out, long long ldo, int out_fp32, const float* conv_w, int taps, const int* row_pos,
+                                const int* row_slot, float* state, long long slot_stride, void* stream_) {
+  cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
+  LP_REQUIRE(x != nullptr && y != nullptr && gain != nullptr && M >= 0 && D > 0, "lp_post_norm_f32: bad arguments");
+  LP_REQUIRE(conv_w == nullptr || (out != nullptr && taps >= 1), "lp_post_norm_f32: a convolution without its operand");
+  LP_REQUIRE(conv_w == nullptr || taps == 1 ||
+                 (row_pos != nullptr && row_slot != nullptr && state != nullptr && slot_stride >= (long long)(taps - 1) * D),
+             "lp_post_norm_f32: no room for the carried inputs");
+  LP_REQUIRE(out != x, "lp_post_norm_f32: the operand needs memory of its own");
+  if (M == 0) return 0;
+  const bool v4 = vec4_ok(D, {x, y, gain, out, conv_w, state}, {ldx, ldy, out != nullptr ? ldo : 0, state != nullptr ? slot_stride : 0});
+  int threads = (v4 ? D / 4 : D);
+  threads = threads >= POST_THREADS ? POST_THREADS : (threads + 31) / 32 * 32;
+  if (out_fp32 && v4)
+    post_norm_kernel<float, 4><<<M, threads, 0, stream>>>(x, ldx, y, ldy, alpha, D, gain, eps, reinterpret_cast<float*>(out), ldo, conv_w, taps,
+                                                          row_pos, row_slot, state, slot_stride);
+  else if (out_fp32)
+    post_norm_kernel<float, 1><<<M, threads, 0, stream>>>(x, ldx, y, ldy, alpha, D, gain, eps, reinterpret_cast<float*>(out), ldo, conv_w, taps,
+                                                          row_pos, row_slot, state, slot_stride);
+  else if (v4)
+    post_norm_kernel<bf16, 4><<<M, threads, 0, stream>>>(x, ldx, y, ldy, alpha, D, gain, eps, reinterpret_cast<bf16*>(out), ldo, conv_w, taps,
+                                                         row_pos, row_slot, state, slot_stride);
+  else
+    post_norm_kernel<bf16, 1><<<M, threads, 0, stream>>>(x, ldx, y, ldy, alpha, D, gain, eps, reinterpret_cast<bf16*>(out), ldo, conv_w, taps,
+                                                         row_pos, row_slot, state, slot_stride);
+  note_launch();
+  LP_CHECK_CUDA(cudaGetLastError());
+  return 0;
+}
 
 extern "C" int lp_add_positions_f32(float* x, long long ldx, int R, int D, const int* row_pos, const float* freq, void* stream_) {
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
@@ -364,7 +633,8 @@ extern "C" int lp_glu_scaled_f32(const void* in, long long ldi, int in_fp32, voi
                                  float a, float b, const float* row_scale, void* stream_) {
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
   LP_REQUIRE(in != nullptr && out != nullptr && M >= 0 && N > 0, "lp_glu_f32: bad arguments");
-  LP_REQUIRE(mode == LP_EPI_XIELU || mode == LP_EPI_SILU_GATE || mode == LP_EPI_RELU2 || mode == LP_EPI_CLAMP_GLU,
+  LP_REQUIRE(mode == LP_EPI_XIELU || mode == LP_EPI_SILU_GATE || mode == LP_EPI_RELU2 || mode == LP_EPI_CLAMP_GLU ||
+                 mode == LP_EPI_GELU_GATE,
              "lp_glu_f32: mode %d is not an activation", mode);
   if (M == 0) return 0;
   const unsigned grid = (unsigned)(((long long)M * N + 255) / 256);

@@ -4,8 +4,9 @@
 // parameter of lp_window_attn_desc:
 //   visibility   window (tokens j with 0 <= i - j < window), keep_first (the request's first tokens stay visible), pool (every block
 //                of P tokens that lies wholly before the window is seen as ONE key / value, the mean of its cached rows)
-//   scores       scale, softcap * tanh(score / softcap), sink (softmax denominator + 1)
-//   projections  RMS norm of q and k per head or over the whole projection, rotation of the first rot_dims dimensions of q and k,
+//   scores       scale, softcap * tanh(score / softcap), sink (softmax denominator + 1), a distance bias per head: after the cap
+//                dist_amp[h] * ln(1 + dist_rate[h] * (i - j)) is taken off
+//   projections  RMS norm of q and k per head or over the whole projection, a temperature per query head (q_temp), rotation of the first rot_dims dimensions of q and k,
 //                optional rotation of the values by their own position with the head output turned back by the query's position
 //                (the weighted sum then depends on the distances i - j only)
 //
@@ -47,6 +48,7 @@ struct WinArgs {
   const float* q_bias; const float* k_bias; const float* v_bias; int v_norm;
   const float* talk; int g_off;
   int chunk, kv_shared;
+  const float* q_temp; const float* dist_amp; const float* dist_rate;
 };
 
 __device__ __forceinline__ float* win_token_row(const WinArgs& a, int seq, int pos) {
@@ -56,6 +58,13 @@ __device__ __forceinline__ float* win_token_row(const WinArgs& a, int seq, int p
 __device__ __forceinline__ float* win_block_row(const WinArgs& a, int seq, int block) {
   const int page = a.pooled_table[(long long)seq * a.max_pooled_pages + block / a.page_size];
   return a.pooled + ((long long)page * a.page_size + block % a.page_size) * (long long)(a.kv_heads * (a.dim + a.vdim));
+}
+
+// what is taken off a score at distance d >= 0: amp ln(1 + rate d).  `exact`: the accurate logarithm (fp32 results); else the fast
+// one, whose absolute error of a few 1e-7 is far below the rounding of a 16-bit output.
+__device__ __forceinline__ float win_distance_bias(float amp, float rate, int d, bool exact) {
+  const float x = fmaf(rate, (float)(d > 0 ? d : 0), 1.0f);
+  return amp * (exact ? logf(x) : __logf(x));
 }
 
 // the two members of rotation pair i
@@ -163,6 +172,7 @@ window_attn_prep_kernel(WinArgs a, int R, const int* __restrict__ row_seq, const
       rinv = 1.0f / sqrtf(s_ss[units + (is_q ? 0 : 1)] / (float)((is_q ? a.heads : a.kv_heads) * a.dim) + a.eps);
       gain = (is_q ? a.q_gain : a.k_gain) + hl * a.dim;
     }
+    if (is_q && a.q_temp != nullptr) rinv *= a.q_temp[hl];      // the head's temperature scales its query
     if (e < half) {
       int d0, d1;
       win_pair(a.rot_layout, half, e, d0, d1);
@@ -224,7 +234,7 @@ window_attn_pool_kernel(WinArgs a, int n_seqs, const int* __restrict__ seq_row0,
   win_block_row(a, s, b)[c] = sum / (float)a.pool;
 }
 
-template <int QH, int NV>
+template <int QH, int NV, bool DIST>
 __global__ void __launch_bounds__(256)
 window_attn_kernel(WinArgs a, int R, const int* __restrict__ row_seq, const int* __restrict__ row_pos, void* __restrict__ out, long long ldo,
                    int out_fp32) {
@@ -249,9 +259,11 @@ window_attn_kernel(WinArgs a, int R, const int* __restrict__ row_seq, const int*
   const int v_off = a.kv_heads * a.dim + g * a.vdim;
   const bool vec = (a.dim % 4 == 0) && (a.vdim % 4 == 0);      // rows and head offsets are then 16-byte aligned
   const bool quads = vec && (a.dim % 16 == 0);
-  float mx[QH], den[QH], acc[QH][NV];
+  float mx[QH], den[QH], acc[QH][NV], amp[QH], rate[QH];
 #pragma unroll
   for (int h = 0; h < QH; ++h) {
+    amp[h] = DIST ? a.dist_amp[h0 + h] : 0.f;
+    rate[h] = DIST ? a.dist_rate[h0 + h] : 0.f;
     // the sink is a key of score 0 without a value: warp 0 starts from it
     mx[h] = (a.sink && warp == 0) ? 0.f : -INFINITY;
     den[h] = (a.sink && warp == 0) ? 1.f : 0.f;
@@ -328,10 +340,12 @@ window_attn_kernel(WinArgs a, int R, const int* __restrict__ row_seq, const int*
       }
     }
     float corr[QH];
+    const int dist = pos - (t < vis.n_keep ? t : vis.lo + (t - vis.n_keep));      // a distance bias comes without pooled blocks
 #pragma unroll
     for (int h = 0; h < QH; ++h) {
       float s = sc[h] * a.scale;
       if (a.softcap > 0.f) s = a.softcap * tanhf(s / a.softcap);
+      if (DIST) s -= win_distance_bias(amp[h], rate[h], dist, out_fp32);
       if (!valid) s = -INFINITY;
       float top = s;
 #pragma unroll
@@ -432,7 +446,7 @@ window_attn_kernel(WinArgs a, int R, const int* __restrict__ row_seq, const int*
 // every (row, key) pair is masked by the row's own rule, so a row's result is the same as in the one-row kernel up to the order of
 // the sums.  A key can stand in the union twice (as a kept token of a late row and as a window token of an early one); each row
 // sees exactly one of the two.
-template <int QH, int NV, int RQ>
+template <int QH, int NV, int RQ, bool DIST>
 __global__ void __launch_bounds__(128)
 window_attn_tile_kernel(WinArgs a, int n_chunks, const int* __restrict__ chunk_seq, const int* __restrict__ chunk_row0,
                         const int* __restrict__ chunk_len, int tiles_per_chunk, const int* __restrict__ row_pos, void* __restrict__ out,
@@ -477,7 +491,12 @@ window_attn_tile_kernel(WinArgs a, int n_chunks, const int* __restrict__ chunk_s
   uni.count = uni.n_keep + uni.n_blocks + (pos0 + nrows - 1 - uni.lo + 1);
   const int v_off = a.kv_heads * a.dim + g * a.vdim;
   const bool quads = (a.dim % 16 == 0) && (a.vdim % 4 == 0);
-  float mx[X], den[X], acc[X][NV];
+  float mx[X], den[X], acc[X][NV], amp[QH], rate[QH];
+#pragma unroll
+  for (int h = 0; h < QH; ++h) {
+    amp[h] = DIST ? a.dist_amp[h0 + h] : 0.f;
+    rate[h] = DIST ? a.dist_rate[h0 + h] : 0.f;
+  }
 #pragma unroll
   for (int x = 0; x < X; ++x) {
     mx[x] = (a.sink && warp == 0) ? 0.f : -INFINITY;
@@ -567,6 +586,7 @@ window_attn_tile_kernel(WinArgs a, int n_chunks, const int* __restrict__ chunk_s
       else seen = seen && idx >= r_lo[rq] && idx <= pos0 + rq;
       float s = sc[x] * a.scale;
       if (a.softcap > 0.f) s = a.softcap * tanhf(s / a.softcap);
+      if (DIST) s -= win_distance_bias(amp[x % QH], rate[x % QH], pos0 + rq - idx, out_fp32);
       if (!seen) s = -INFINITY;
       float top = s;
 #pragma unroll
@@ -1064,6 +1084,9 @@ static int fill_win(WinArgs& a, const lp_window_attn_desc* d, bool need_q) {
   a.scale = d->scale; a.softcap = d->softcap; a.sink = d->sink;
   a.q_bias = d->q_bias; a.k_bias = d->k_bias; a.v_bias = d->v_bias; a.v_norm = d->v_norm;
   a.talk = d->talk; a.g_off = d->g_off;
+  a.q_temp = d->q_temp; a.dist_amp = d->dist_amp; a.dist_rate = d->dist_rate;
+  LP_REQUIRE((d->dist_amp != nullptr) == (d->dist_rate != nullptr), "lp_window_attn: one half of a distance bias without the other");
+  LP_REQUIRE(d->dist_amp == nullptr || d->pool == 0, "lp_window_attn: a distance bias to pooled blocks is not defined");
   return 0;
 }
 
@@ -1074,7 +1097,7 @@ static size_t win_smem_floats(int qh, int w, int dim, int vdim) {
   return 2 * (size_t)w * 32 + (size_t)qh * dim + (size_t)w * qh * 32 + 2 * (size_t)w * qh + (size_t)w * qh * vdim + (size_t)qh * vdim;
 }
 
-template <int QH>
+template <int QH, bool DIST>
 static int launch_window_attn(const WinArgs& a, int R, const int* row_seq, const int* row_pos, void* out, long long ldo, int out_fp32,
                               cudaStream_t stream) {
   int warps = R <= WIN_SPLIT_ROWS ? 8 : 4;
@@ -1083,10 +1106,10 @@ static int launch_window_attn(const WinArgs& a, int R, const int* row_seq, const
   LP_REQUIRE(smem <= 48 * 1024, "lp_window_attn: dim=%d vdim=%d do not fit shared memory", a.dim, a.vdim);
   const dim3 grid(R, a.kv_heads * (a.heads / a.kv_heads / QH));
   const int nv = (a.vdim + 31) / 32;
-  if (nv <= 1) window_attn_kernel<QH, 1><<<grid, warps * 32, smem, stream>>>(a, R, row_seq, row_pos, out, ldo, out_fp32);
-  else if (nv <= 2) window_attn_kernel<QH, 2><<<grid, warps * 32, smem, stream>>>(a, R, row_seq, row_pos, out, ldo, out_fp32);
-  else if (nv <= 4) window_attn_kernel<QH, 4><<<grid, warps * 32, smem, stream>>>(a, R, row_seq, row_pos, out, ldo, out_fp32);
-  else window_attn_kernel<QH, 8><<<grid, warps * 32, smem, stream>>>(a, R, row_seq, row_pos, out, ldo, out_fp32);
+  if (nv <= 1) window_attn_kernel<QH, 1, DIST><<<grid, warps * 32, smem, stream>>>(a, R, row_seq, row_pos, out, ldo, out_fp32);
+  else if (nv <= 2) window_attn_kernel<QH, 2, DIST><<<grid, warps * 32, smem, stream>>>(a, R, row_seq, row_pos, out, ldo, out_fp32);
+  else if (nv <= 4) window_attn_kernel<QH, 4, DIST><<<grid, warps * 32, smem, stream>>>(a, R, row_seq, row_pos, out, ldo, out_fp32);
+  else window_attn_kernel<QH, 8, DIST><<<grid, warps * 32, smem, stream>>>(a, R, row_seq, row_pos, out, ldo, out_fp32);
   note_launch();
   LP_CHECK_CUDA(cudaGetLastError());
   return 0;
@@ -1097,7 +1120,7 @@ static size_t win_tile_smem_floats(int x, int w, int dim, int vdim) {
 }
 
 // 0: launched; 1: the sizes do not fit the tile kernel's shared memory (the caller takes the one-row kernel)
-template <int QH, int RQ>
+template <int QH, int RQ, bool DIST>
 static int launch_window_attn_tiles(const WinArgs& a, int R, int n_chunks, const int* chunk_seq, const int* chunk_row0, const int* chunk_len,
                                     const int* row_pos, void* out, long long ldo, int out_fp32, cudaStream_t stream) {
   int warps = 4;
@@ -1108,9 +1131,9 @@ static int launch_window_attn_tiles(const WinArgs& a, int R, int n_chunks, const
   const int tiles = (longest + RQ - 1) / RQ;
   const dim3 grid(n_chunks * tiles, a.kv_heads * (a.heads / a.kv_heads / QH));
   const int nv = (a.vdim + 31) / 32;
-  if (nv <= 1) window_attn_tile_kernel<QH, 1, RQ><<<grid, warps * 32, smem, stream>>>(a, n_chunks, chunk_seq, chunk_row0, chunk_len, tiles, row_pos, out, ldo, out_fp32);
-  else if (nv <= 2) window_attn_tile_kernel<QH, 2, RQ><<<grid, warps * 32, smem, stream>>>(a, n_chunks, chunk_seq, chunk_row0, chunk_len, tiles, row_pos, out, ldo, out_fp32);
-  else if (nv <= 4) window_attn_tile_kernel<QH, 4, RQ><<<grid, warps * 32, smem, stream>>>(a, n_chunks, chunk_seq, chunk_row0, chunk_len, tiles, row_pos, out, ldo, out_fp32);
+  if (nv <= 1) window_attn_tile_kernel<QH, 1, RQ, DIST><<<grid, warps * 32, smem, stream>>>(a, n_chunks, chunk_seq, chunk_row0, chunk_len, tiles, row_pos, out, ldo, out_fp32);
+  else if (nv <= 2) window_attn_tile_kernel<QH, 2, RQ, DIST><<<grid, warps * 32, smem, stream>>>(a, n_chunks, chunk_seq, chunk_row0, chunk_len, tiles, row_pos, out, ldo, out_fp32);
+  else if (nv <= 4) window_attn_tile_kernel<QH, 4, RQ, DIST><<<grid, warps * 32, smem, stream>>>(a, n_chunks, chunk_seq, chunk_row0, chunk_len, tiles, row_pos, out, ldo, out_fp32);
   else return 1;      // value heads wider than 128 keep too many sums per lane for a tile of rows
   note_launch();
   LP_CHECK_CUDA(cudaGetLastError());
@@ -1161,9 +1184,14 @@ extern "C" int lp_window_attn(const lp_window_attn_desc* d, int R, const int* ro
              WIN_MAX_DIM);
   if (R <= 0) return 0;
   const int ratio = d->heads / d->kv_heads;
-  if (ratio % 4 == 0) return launch_window_attn<4>(a, R, row_seq, row_pos, out, ldo, out_fp32, stream);
-  if (ratio % 2 == 0) return launch_window_attn<2>(a, R, row_seq, row_pos, out, ldo, out_fp32, stream);
-  return launch_window_attn<1>(a, R, row_seq, row_pos, out, ldo, out_fp32, stream);
+  if (d->dist_amp != nullptr) {
+    if (ratio % 4 == 0) return launch_window_attn<4, true>(a, R, row_seq, row_pos, out, ldo, out_fp32, stream);
+    if (ratio % 2 == 0) return launch_window_attn<2, true>(a, R, row_seq, row_pos, out, ldo, out_fp32, stream);
+    return launch_window_attn<1, true>(a, R, row_seq, row_pos, out, ldo, out_fp32, stream);
+  }
+  if (ratio % 4 == 0) return launch_window_attn<4, false>(a, R, row_seq, row_pos, out, ldo, out_fp32, stream);
+  if (ratio % 2 == 0) return launch_window_attn<2, false>(a, R, row_seq, row_pos, out, ldo, out_fp32, stream);
+  return launch_window_attn<1, false>(a, R, row_seq, row_pos, out, ldo, out_fp32, stream);
 }
 
 static int window_attn_talk(const lp_window_attn_desc* d, int R, const int* row_seq, const int* row_pos, const TalkChunks& ch, void* out,
@@ -1172,6 +1200,7 @@ static int window_attn_talk(const lp_window_attn_desc* d, int R, const int* row_
   if (int rc = fill_win(a, d, true)) return rc;
   LP_REQUIRE(out != nullptr && row_seq != nullptr && row_pos != nullptr && d->talk != nullptr, "lp_window_attn_talk: null operand");
   LP_REQUIRE(d->v_inv_freq == nullptr, "lp_window_attn_talk: rotated values are not mixed here");
+  LP_REQUIRE(d->dist_amp == nullptr, "lp_window_attn_talk: a distance bias together with mixed heads is not supported");
   if (R <= 0) return 0;
   const int n_out = d->heads * d->vdim;
   LP_REQUIRE(n_out <= 256 * TALK_MAX_ACC, "lp_window_attn_talk: heads * vdim = %d > %d", n_out, 256 * TALK_MAX_ACC);
@@ -1216,9 +1245,15 @@ extern "C" int lp_window_attn_tiles(const lp_window_attn_desc* d, int R, const i
   if (R <= 0 || n_chunks <= 0) return 0;
   const int ratio = d->heads / d->kv_heads;
   int rc;
-  if (ratio % 4 == 0) rc = launch_window_attn_tiles<4, 2>(a, R, n_chunks, chunk_seq, chunk_row0, chunk_len, row_pos, out, ldo, out_fp32, stream);
-  else if (ratio % 2 == 0) rc = launch_window_attn_tiles<2, 4>(a, R, n_chunks, chunk_seq, chunk_row0, chunk_len, row_pos, out, ldo, out_fp32, stream);
-  else rc = launch_window_attn_tiles<1, 4>(a, R, n_chunks, chunk_seq, chunk_row0, chunk_len, row_pos, out, ldo, out_fp32, stream);
+  if (d->dist_amp != nullptr) {
+    if (ratio % 4 == 0) rc = launch_window_attn_tiles<4, 2, true>(a, R, n_chunks, chunk_seq, chunk_row0, chunk_len, row_pos, out, ldo, out_fp32, stream);
+    else if (ratio % 2 == 0) rc = launch_window_attn_tiles<2, 4, true>(a, R, n_chunks, chunk_seq, chunk_row0, chunk_len, row_pos, out, ldo, out_fp32, stream);
+    else rc = launch_window_attn_tiles<1, 4, true>(a, R, n_chunks, chunk_seq, chunk_row0, chunk_len, row_pos, out, ldo, out_fp32, stream);
+  } else {
+    if (ratio % 4 == 0) rc = launch_window_attn_tiles<4, 2, false>(a, R, n_chunks, chunk_seq, chunk_row0, chunk_len, row_pos, out, ldo, out_fp32, stream);
+    else if (ratio % 2 == 0) rc = launch_window_attn_tiles<2, 4, false>(a, R, n_chunks, chunk_seq, chunk_row0, chunk_len, row_pos, out, ldo, out_fp32, stream);
+    else rc = launch_window_attn_tiles<1, 4, false>(a, R, n_chunks, chunk_seq, chunk_row0, chunk_len, row_pos, out, ldo, out_fp32, stream);
+  }
   if (rc == 1) return lp_window_attn(d, R, row_seq, row_pos, out, ldo, out_fp32, stream_);
   return rc;
 }

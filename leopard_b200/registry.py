@@ -60,6 +60,11 @@ def _kamosun(path, **kw):
     return kamosun.load(path, **kw)
 
 
+def _komazen(path, **kw):
+    from . import komazen
+    return komazen.load(path, **kw)
+
+
 def _llava(path, **kw):
     from .hf import myLlavaForConditionalGeneration
     return myLlavaForConditionalGeneration.from_pretrained(path, **kw)
@@ -69,6 +74,7 @@ register("Zudalorn", _zudalorn)
 register("Ronelorn", _ronelorn)
 register("Gavatar", _gavatar)
 register("Kamosun", _kamosun)
+register("Komazen", _komazen)
 register("LlavaForConditionalGeneration", _llava)
 register("myLlavaForConditionalGeneration", _llava)
 register("llava", _llava)

@@ -4,9 +4,9 @@ A model is a `SeqLMConfig`: vocabulary, width, norm epsilon and style, and a tup
 (`RetentionConfig`, `LatentAttentionConfig`, `WindowAttentionConfig`, `MinGRUConfig`, `MLSTMConfig`, or a `ParallelMixerConfig` of
 two of them side by side) and its feed-forward
 (`DenseFFConfig`, `MoEConfig` or none); a layer may run on another layer's weights with a cache or state of its own (a looped stack
-is such a list), shift its mixer's input towards the previous token's, and add a learned vector to the stream before it runs.  Every mechanism is a
-separate native entry point with its constants as arguments (include/leopard_b200.h, "32-BIT RESIDUAL-STREAM MODELS"), so another
-design is another list.  The residual stream, norms, routers, rotary angles, attention scores and recurrent state are fp32; matrix
+is such a list), shift its mixer's input towards the previous token's, run a short causal convolution over the input of its
+sublayers, and add a learned vector to the stream before it runs.  Every mechanism is a separate native entry point with its constants
+as arguments (include/leopard_b200.h, "32-BIT RESIDUAL-STREAM MODELS"), so another design is another list.  The residual stream, norms, routers, rotary angles, attention scores and recurrent state are fp32; matrix
 products take bf16 weights and, in the serving precision, bf16 activations with fp32 accumulation ("bfloat16"), or fp32 activations
 on fp32 FMAs ("float32": a true 32-bit forward, no tensor-core rounding).
 
@@ -130,6 +130,10 @@ class LatentAttentionConfig:
     q_rank: int = 0                # > 0: queries go through a normed latent of this size (mix.dq, mix.dq.norm, mix.uq) instead of mix.q
     sink: bool = False             # exp(mix.sink[h]) joins head h's softmax denominator
     head_gate: bool = False        # head h's output is multiplied by sigmoid(mix.g h)[h]
+    out_gate: bool = False         # the concatenated heads are multiplied element by element by sigmoid(mix.g h)
+    # the layer has no mix.dkv: it reads the latents and rotated key parts that layer cached (earlier in the same step) with its own
+    # mix.uk, mix.uv, queries, window and everything else
+    kv_from: Optional[int] = None
 
 
 @dataclass(frozen=True)
@@ -158,6 +162,8 @@ class WindowAttentionConfig:
     # the layer has no key / value tensors: it reads the cache rows of that layer (keys after norm and rotation, values), written
     # earlier in the same step, with its own queries, visibility and everything else
     kv_from: Optional[int] = None
+    head_temp: bool = False        # head h's scores are multiplied by mix.temp[h]
+    distance_bias: bool = False    # mix.r1[h] * ln(1 + mix.r2[h] * (i - j)) is taken off head h's score (after the cap)
 
 
 @dataclass(frozen=True)
@@ -190,7 +196,8 @@ GLU_SLOPE = 1.702                  # the sigmoid's slope in the clamped gated un
 @dataclass(frozen=True)
 class DenseFFConfig:
     ff: int
-    # "xielu" (two learned constants in mlp.act), "relu2" (the square of relu), or "clamp_glu": with g = min(mlp.gate h, limit) and
+    # "xielu" (two learned constants in mlp.act), "relu2" (the square of relu), "gelu_glu" (gelu(mlp.gate h) * mlp.up h, gelu in its
+    # tanh form), or "clamp_glu": with g = min(mlp.gate h, limit) and
     # u = clamp(mlp.up h, -limit, limit) the hidden vector is g sigmoid(1.702 g) (u + 1)
     act: str = "xielu"
     limit: float = 0.0
@@ -222,6 +229,10 @@ class LayerConfig:
     # the mixer reads h_t + (h_(t-1) - h_t) * shift per channel instead of h_t (h: the normed stream; the previous token's h is part of
     # the request's state, zeros before the first token); the vector is the layer's tensor `shift`
     token_shift: bool = False
+    # > 0: what each sublayer reads, h, becomes h + conv(h), a causal convolution of that many taps over time on each channel (tensors conv1
+    # for the mixer, conv2 for the feed-forward, [width, taps], the current token's tap last); the last taps - 1 inputs are part of
+    # the request's state, zeros before the first token
+    input_conv: int = 0
     add_before: Optional[Tuple[str, int]] = None   # (tensor, row): that row is added to the stream right before this layer runs
 
 
@@ -235,9 +246,12 @@ class SeqLMConfig:
     # "sandwich": x <- x + norm_b(sublayer(norm_a(x))), every norm with ONE gain; "pre": x <- x + residual_mult * sublayer(norm(x)),
     # the norm's gain a vector stored around zero (x / rms * (1 + w)); "sandwich_vector": the sandwich form with such vector gains;
     # "parallel_dyt": x <- x + residual_mult * (mixer(norm1(x)) + ff(norm2(x))), both sublayers on the same x, every norm (the final
-    # one too) a Dynamic Tanh tanh(alpha x) * w + b with the tensors <name>, <name>.alpha, <name>.b
+    # one too) a Dynamic Tanh tanh(alpha x) * w + b with the tensors <name>, <name>.alpha, <name>.b; "post": the norm comes after the sum,
+    # x <- norm1(post_alpha * x + mixer(x)), then x <- norm2(post_alpha * x + ff(x)), the sublayers read x itself and every norm has a
+    # plain vector gain (x / rms * w)
     norm: str = "sandwich"
     residual_mult: float = 1.0
+    post_alpha: float = 1.0
     embed_scale: float = 1.0
     # > 0: absolute sinusoidal positions are added to the embedding, entries (2i, 2i + 1) = (sin, cos)(p * base^(-2i / width))
     position_base: float = 0.0
@@ -261,7 +275,8 @@ def softplus(x: float) -> float:
 # ---------------------------------------------------------------------------------------------------------------- weights
 class SeqLMWeights:
     """Device tensors in the layout the kernels read.  `get(name)` returns a checkpoint tensor; `name(layer, key)` maps the generic
-    keys used here (norm1, norm1b, norm2, norm2b, mix.*, mlp.*; embed, final.norm, head with layer None) to checkpoint names."""
+    keys used here (norm1, norm1b, norm2, norm2b, conv1, conv2, mix.*, mlp.*; embed, final.norm, head with layer None) to checkpoint
+    names."""
 
     def __init__(self, cfg: SeqLMConfig, get: Callable[[str], torch.Tensor], name: Callable[[Optional[int], str], str], device):
         self.cfg, self.device = cfg, torch.device(device)
@@ -285,10 +300,15 @@ class SeqLMWeights:
         def one_plus(layer, key):           # a gain stored around zero
             return (1.0 + w(layer, key, (cfg.width,)).float()).contiguous().to(dev)
 
-        if cfg.norm not in ("sandwich", "pre", "sandwich_vector", "parallel_dyt"):
+        if cfg.norm not in ("sandwich", "pre", "sandwich_vector", "parallel_dyt", "post"):
             raise ValueError(f"unknown norm style {cfg.norm!r}")
         pre = cfg.norm == "pre"
         dyt = cfg.norm == "parallel_dyt"
+        post = cfg.norm == "post"
+        if post and any(lc.token_shift or lc.add_before is not None for lc in cfg.layers):
+            raise ValueError("token shift and added vectors do not go with the post-norm layer form")
+        if dyt and any(lc.input_conv for lc in cfg.layers):
+            raise ValueError("input convolutions do not go with the parallel layer form")
         if (cfg.residual_gate or cfg.depth_average) and not dyt:
             raise ValueError("gated residual branches and the depth average belong to the parallel layer form")
         vector = cfg.norm != "sandwich"
@@ -299,7 +319,7 @@ class SeqLMWeights:
         D = cfg.width
         self.embed = mat(w(None, "embed", (cfg.vocab, D)))
         self.head = mat(w(None, "head", (cfg.vocab, D)))
-        self.final_gain = dyt_norm(None, "final.norm") if dyt else one_plus(None, "final.norm") if vector else num(None, "final.norm")
+        self.final_gain = dyt_norm(None, "final.norm") if dyt else vec(w(None, "final.norm", (D,))) if post else one_plus(None, "final.norm") if vector else num(None, "final.norm")
         if cfg.position_base > 0:      # frequencies in float64, split into two floats hi + lo
             f64 = cfg.position_base ** (-2.0 * np.arange((D + 1) // 2, dtype=np.float64) / D)
             hi = f64.astype(np.float32)
@@ -322,12 +342,14 @@ class SeqLMWeights:
                 j = lc.weights_of
                 if not 0 <= j < len(cfg.layers) or cfg.layers[j].weights_of is not None:
                     raise ValueError(f"layer {i}: weights_of = {j} must name a layer that has tensors of its own")
-                if (cfg.layers[j].mixer, cfg.layers[j].ff, cfg.layers[j].token_shift) != (lc.mixer, lc.ff, lc.token_shift):
+                if any(getattr(cfg.layers[j], k) != getattr(lc, k) for k in ("mixer", "ff", "token_shift", "input_conv")):
                     raise ValueError(f"layer {i} differs from layer {j}, whose weights it uses")
                 self.layers.append(None)              # linked below, once every owner is loaded
                 continue
             if dyt:
                 lw: Dict[str, object] = {"norm1": dyt_norm(i, "norm1")}
+            elif post:
+                lw = {"norm1": vec(w(i, "norm1", (D,)))}
             elif pre:
                 lw = {"norm1": one_plus(i, "norm1")}
             elif vector:
@@ -336,6 +358,9 @@ class SeqLMWeights:
                 lw = {k: num(i, k) for k in ("norm1", "norm1b")}
             if lc.token_shift:
                 lw["shift"] = vec(w(i, "shift", (D,)))
+            if lc.input_conv:      # [taps][width]: the lanes of a kernel read neighbouring channels of one tap
+                for k in ("conv1", "conv2") if lc.ff is not None else ("conv1",):
+                    lw[k] = vec(w(i, k, (D, lc.input_conv)).t())
             def mixer_weights(m, pfx: str) -> Dict[str, object]:
                 """the tensors of one mixer, named <pfx><key> in the checkpoint"""
                 mw: Dict[str, object] = {}
@@ -372,6 +397,12 @@ class SeqLMWeights:
                         mw["talk"] = vec(w(i, pfx + "talk", (m.heads, m.heads)))
                     elif m.out_gate:      # the gate rides on the mixing kernel: no mixing is the unit matrix
                         mw["talk"] = torch.eye(m.heads, dtype=F32).to(dev)
+                    if m.head_temp:
+                        mw["temp"] = vec(w(i, pfx + "temp", (m.heads,)))
+                    if m.distance_bias:
+                        if m.pool or m.talking_heads or m.out_gate:
+                            raise ValueError(f"layer {i}: a distance bias with pooled blocks or with mixed or gated heads is not supported")
+                        mw["dist_amp"], mw["dist_rate"] = vec(w(i, pfx + "r1", (m.heads,))), vec(w(i, pfx + "r2", (m.heads,)))
                     if (m.talking_heads or m.out_gate) and m.value_rot is not None:
                         raise ValueError(f"layer {i}: mixed or gated heads with rotated values are not supported")
                     if m.qk_norm == "head":      # a layer without keys of its own hands the kernel its query gain twice (the second is unused)
@@ -398,18 +429,23 @@ class SeqLMWeights:
                         raise ValueError(f"layer {i}: unknown retention form {m.form!r}")
                 else:
                     per = m.dim + m.rot_dim
-                    # one product of h: [queries or their latent | key / value latent (+ shared rotated key) | one gate per head]
-                    parts = [w(i, pfx + "dq", (m.q_rank, D)) if m.q_rank else w(i, pfx + "q", (m.heads * per, D)),
-                             w(i, pfx + "dkv", (m.kv_rank + m.rot_dim, D))]
-                    if m.head_gate:
-                        parts.append(w(i, pfx + "g", (m.heads, D)))
+                    # one product of h: [queries or their latent | key / value latent (+ shared rotated key), when the layer has its own |
+                    # one gate per head, or one per output element]
+                    parts = [w(i, pfx + "dq", (m.q_rank, D)) if m.q_rank else w(i, pfx + "q", (m.heads * per, D))]
+                    if m.kv_from is None:
+                        parts.append(w(i, pfx + "dkv", (m.kv_rank + m.rot_dim, D)))
+                    if m.head_gate and m.out_gate:
+                        raise ValueError(f"layer {i}: latent attention has one kind of gate")
+                    if m.head_gate or m.out_gate:
+                        parts.append(w(i, pfx + "g", (m.heads if m.head_gate else m.heads * m.vdim, D)))
                     mw["w_qdkv"] = mat(torch.cat(parts, 0))
                     if m.q_rank:
                         mw["cq_gain"] = vec(w(i, pfx + "dq.norm", (m.q_rank,)))
                         mw["w_uq"] = mat(w(i, pfx + "uq", (m.heads * per, m.q_rank)))
                     if m.sink:
                         mw["sink"] = vec(w(i, pfx + "sink", (m.heads,)))
-                    mw["c_gain"] = w(i, pfx + "dkv.norm", (m.kv_rank,)).float().contiguous().to(dev)
+                    if m.kv_from is None:
+                        mw["c_gain"] = vec(w(i, pfx + "dkv.norm", (m.kv_rank,)))
                     uk = w(i, pfx + "uk", (m.heads * m.dim, m.kv_rank))
                     mw["w_ukT"] = mat(uk.reshape(m.heads, m.dim, m.kv_rank).transpose(1, 2))       # [heads][kv_rank, dim]
                     mw["w_uv"] = mat(w(i, pfx + "uv", (m.heads * m.vdim, m.kv_rank)))                 # [heads][vdim, kv_rank]
@@ -447,9 +483,9 @@ class SeqLMWeights:
                 lw["dwa"] = vec(w(i, "dwa", (i + 2,)))
             f = lc.ff
             if f is not None:
-                lw.update({"norm2": dyt_norm(i, "norm2")} if dyt else {"norm2": one_plus(i, "norm2")} if pre else
+                lw.update({"norm2": dyt_norm(i, "norm2")} if dyt else {"norm2": vec(w(i, "norm2", (D,)))} if post else {"norm2": one_plus(i, "norm2")} if pre else
                           {k: (one_plus(i, k) if vector else num(i, k)) for k in ("norm2", "norm2b")})
-            if isinstance(f, DenseFFConfig) and f.act == "clamp_glu":
+            if isinstance(f, DenseFFConfig) and f.act in ("clamp_glu", "gelu_glu"):
                 lw["w_gu"] = mat(torch.cat([w(i, "mlp.gate", (f.ff, D)), w(i, "mlp.up", (f.ff, D))], 0))
                 lw["w_down"] = mat(w(i, "mlp.down", (D, f.ff)))
             elif isinstance(f, DenseFFConfig):
@@ -522,6 +558,7 @@ class _Batch:
         R = sum(lens)
         self.R, self.n, self.lens = R, n, lens
         self.decode = all(ln == 1 for ln in lens)
+        self.longest_chunk = min(max(lens), _lib.RETENTION_CHUNK)
         row0 = np.zeros(n + 1, np.int32)
         row0[1:] = np.cumsum(lens)
         pos0 = np.array([s.length for s in seqs], np.int32)
@@ -606,29 +643,31 @@ class SeqLMEngine:
         # what every mixer keeps per request: rows of a paged cache (attention), rows of a summary pool (pooled blocks), a state.
         # The tables are keyed by the layer, or by (layer, "left" | "right") for the branches of a parallel mixer.
         rows, states, summaries, looks, keep = [], [], [], [], 0
-        self._cache_index, self._state_index, self._summary_index, self._shift_index = {}, {}, {}, []
+        self._cache_index, self._state_index, self._summary_index, self._shift_index, self._conv_index = {}, {}, {}, [], {}
 
         def look_back(m):      # how far back a windowed or block-local layer reads (None: everything)
-            bounds = [v for v in (m.window, m.chunk) if v and v > 0]
+            bounds = [v for v in (m.window, getattr(m, "chunk", None)) if v and v > 0]
             return min(bounds) if bounds else None
 
         def claim(key, m):
             nonlocal keep
             ci = si = pi = -1
-            if isinstance(m, LatentAttentionConfig):
-                ci = len(rows)
-                rows.append(m.kv_rank + m.rot_dim)
-                looks.append(m.window if m.window and m.window > 0 else None)
-            elif isinstance(m, WindowAttentionConfig) and m.kv_from is not None:
+            if getattr(m, "kv_from", None) is not None:
                 j = m.kv_from
                 src = cfg.layers[j].mixer if 0 <= j < len(cfg.layers) and not isinstance(key, tuple) and j < key else None
-                if not isinstance(src, WindowAttentionConfig) or src.kv_from is not None:
-                    raise ValueError(f"layer {key}: kv_from = {j} must name an earlier attention layer that has keys and values of its own")
-                if (src.kv_heads, src.dim, src.vdim, src.rot) != (m.kv_heads, m.dim, m.vdim, m.rot) or m.pool or src.value_rot or m.value_rot:
+                if type(src) is not type(m) or src.kv_from is not None:
+                    raise ValueError(f"layer {key}: kv_from = {j} must name an earlier attention layer of its kind that has keys and values of its own")
+                same = ("kv_rank", "rot_dim", "rot") if isinstance(m, LatentAttentionConfig) else ("kv_heads", "dim", "vdim", "rot")
+                if any(getattr(src, k) != getattr(m, k) for k in same) or (
+                        isinstance(m, WindowAttentionConfig) and (m.pool or src.value_rot or m.value_rot)):
                     raise ValueError(f"layer {key}: its key / value sizes and rotation differ from those of layer {j}, whose cache it reads")
                 ci = self._cache_index[j]
                 looks.append(look_back(m))      # the owner's rows must stay for as long as this layer looks back
-                keep = max(keep, m.keep_first if look_back(m) else 0)
+                keep = max(keep, getattr(m, "keep_first", 0) if looks[-1] else 0)
+            elif isinstance(m, LatentAttentionConfig):
+                ci = len(rows)
+                rows.append(m.kv_rank + m.rot_dim)
+                looks.append(look_back(m))
             elif isinstance(m, WindowAttentionConfig):
                 ci = len(rows)
                 rows.append(m.kv_heads * (m.dim + m.vdim))
@@ -656,6 +695,12 @@ class SeqLMEngine:
             self._shift_index.append(len(states) if lc.token_shift else -1)
             if lc.token_shift:
                 states.append((cfg.width,))
+            if lc.input_conv and lc.input_conv > int(self.L.lp_causal_conv_max_taps()):
+                raise ValueError(f"layer {li}: a convolution of {lc.input_conv} taps is not built")
+            for which in ("conv1", "conv2") if lc.ff is not None else ("conv1",):
+                if lc.input_conv > 1:      # the last taps - 1 inputs of the mixer and of the feed-forward
+                    self._conv_index[(li, which)] = len(states)
+                    states.append((lc.input_conv - 1, cfg.width))
             if isinstance(lc.mixer, ParallelMixerConfig):
                 claim((li, "left"), lc.mixer.left)
                 claim((li, "right"), lc.mixer.right)
@@ -737,12 +782,14 @@ class SeqLMEngine:
         self._check(self.L.lp_linear(C.byref(d), self._stream()), "lp_linear")
         return out
 
-    def linear_heads(self, a: torch.Tensor, a_head: int, w: torch.Tensor, out: torch.Tensor, out_head: int):
-        """Per head h: out[:, h*out_head : +N] = a[:, h*a_head : +K] @ w[h].T with w [heads, N, K]."""
+    def linear_heads(self, a: torch.Tensor, a_head: int, w: torch.Tensor, out: torch.Tensor, out_head: int, gate=None):
+        """Per head h: out[:, h*out_head : +N] = a[:, h*a_head : +K] @ w[h].T with w [heads, N, K]; gate (fp32 rows, N per head): the
+        result is multiplied by its sigmoid."""
         heads, N, K = w.shape
         d = _lib.LinearDesc(A=_lib.ptr(a), lda=a.stride(0), a_batch=a_head, a_fp32=int(a.dtype == F32), W=_lib.ptr(w), ldw=w.stride(1),
                             w_batch=w.stride(0), C=_lib.ptr(out), ldc=out.stride(0), c_batch=out_head, c_fp32=int(out.dtype == F32),
-                            M=a.shape[0], N=N, K=K, batch=heads, epi=_lib.EPI_NONE, epi_a=0.0, epi_b=0.0)
+                            M=a.shape[0], N=N, K=K, batch=heads, epi=_lib.EPI_NONE, epi_a=0.0, epi_b=0.0, gate=_lib.ptr(gate),
+                            ldg=gate.stride(0) if gate is not None else 0, gate_batch=N)
         self._check(self.L.lp_linear(C.byref(d), self._stream()), "lp_linear")
         return out
 
@@ -769,6 +816,28 @@ class SeqLMEngine:
                                int(self.act == F32), self._stream())
         self._check(rc, "lp_dyt_f32")
         return out, out2
+
+    def convolved(self, h: torch.Tensor, li: int, which: str, b: _Batch) -> torch.Tensor:
+        """h + conv(h) in the operand dtype for the sublayer `which` of layer li (h: fp32 rows); its carried inputs move on"""
+        taps, w = self.cfg.layers[li].input_conv, self.w.layers[li][which]
+        out = self._empty(h.shape, self.act)
+        state = self._conv_state(li, which)
+        rc = self.L.lp_causal_conv_f32(_lib.ptr(h), h.stride(0), _lib.ptr(w), taps, h.shape[1], b.n_chunks, _lib.ptr(b.chunk_seq),
+                                       _lib.ptr(b.chunk_row0), _lib.ptr(b.chunk_len), b.longest_chunk, _lib.ptr(b.row_pos),
+                                       _lib.ptr(b.seq_row0), _lib.ptr(b.seq_slot), _lib.ptr(state), state.stride(0) if state is not None else 0,
+                                       _lib.ptr(out), out.stride(0), int(out.dtype == F32), self._stream())
+        self._check(rc, "lp_causal_conv_f32")
+        return out
+
+    def _conv_state(self, li: int, which: str) -> Optional[torch.Tensor]:
+        j = self._conv_index.get((li, which))
+        return self.cache.states[j] if j is not None else None
+
+    def operand(self, x: torch.Tensor, gain, li: int, which: str, b: _Batch) -> torch.Tensor:
+        """what a sublayer of a layer with norms ahead of it reads: the normed stream, convolved when the layer says so"""
+        if self.cfg.layers[li].input_conv:
+            return self.convolved(self.norm(x, gain, F32), li, which, b)
+        return self.norm(x, gain, self.act)
 
     # ------------------------------------------------------------------ mixers
     def _retention(self, li, m: RetentionConfig, lw, h: torch.Tensor, b: _Batch, into=None, proj=None) -> torch.Tensor:
@@ -806,20 +875,22 @@ class SeqLMEngine:
         per = m.dim + m.rot_dim
         qd = proj if proj is not None else self.linear(h, lw["w_qdkv"], F32)
         nq = m.q_rank or m.heads * per
-        dkv = qd[:, nq: nq + m.kv_rank + m.rot_dim]
-        gate = qd[:, nq + m.kv_rank + m.rot_dim:] if m.head_gate else None
+        nkv = m.kv_rank + m.rot_dim if m.kv_from is None else 0      # a layer on another layer's latents brings none
+        dkv = qd[:, nq: nq + nkv] if nkv else None
+        head_gate = qd[:, nq + nkv:] if m.head_gate else None
+        out_gate = qd[:, nq + nkv:] if m.out_gate else None
         if m.q_rank:      # queries through their own normed latent
             q = self.linear(self.norm(qd[:, :nq], lw["cq_gain"], self.act), lw["w_uq"], F32)
         else:
             q = qd[:, :nq]
         pool = self.cache.pools[self._cache_index[li]]
         d = _lib.LatentDesc(q=_lib.ptr(q), ldq=q.stride(0), dkv=_lib.ptr(dkv), lddkv=qd.stride(0), heads=m.heads, dim=m.dim,
-                            rot_dim=m.rot_dim, kv_rank=m.kv_rank, c_gain=_lib.ptr(lw["c_gain"]), eps=self.cfg.eps,
+                            rot_dim=m.rot_dim, kv_rank=m.kv_rank, c_gain=_lib.ptr(lw.get("c_gain")), eps=self.cfg.eps,
                             inv_freq=_lib.ptr(lw["inv_freq"]), rot_dims=m.rot.dims,
                             rot_layout=_lib.ROT_INTERLEAVED if m.rot.layout == "interleaved" else _lib.ROT_HALF,
                             rot_mscale=lw["rot_mag"], cache=_lib.ptr(pool), page_size=self.cache.page_size,
                             page_table=_lib.ptr(b.page_table), max_pages=b.max_pages, window=m.window or 0, scale=m.scale,
-                            sink=_lib.ptr(lw.get("sink")), gate=_lib.ptr(gate), ldg=qd.stride(0) if gate is not None else 0)
+                            sink=_lib.ptr(lw.get("sink")), gate=_lib.ptr(head_gate), ldg=qd.stride(0) if head_gate is not None else 0)
         self._check(self.L.lp_latent_prep(C.byref(d), b.R, _lib.ptr(b.row_seq), _lib.ptr(b.row_pos), self._stream()), "lp_latent_prep")
         q_abs = self._empty((b.R, m.heads * m.kv_rank), F32)
         self.linear_heads(q, per, lw["w_ukT"], q_abs, m.kv_rank)
@@ -828,7 +899,7 @@ class SeqLMEngine:
                                      _lib.ptr(lat), lat.stride(0), int(lat.dtype == F32), self._stream())
         self._check(rc, "lp_latent_attend")
         o = self._empty((b.R, m.heads * m.vdim), self.act)
-        self.linear_heads(lat, m.kv_rank, lw["w_uv"].view(m.heads, m.vdim, m.kv_rank), o, m.vdim)
+        self.linear_heads(lat, m.kv_rank, lw["w_uv"].view(m.heads, m.vdim, m.kv_rank), o, m.vdim, gate=out_gate)
         return self.linear(o, lw["w_o"], F32, into=into)
 
     def _window_attention(self, li, m: WindowAttentionConfig, lw, h: torch.Tensor, b: _Batch, into=None, proj=None) -> torch.Tensor:
@@ -857,7 +928,8 @@ class SeqLMEngine:
             pooled_table=_lib.ptr(b.summary_table[stream]) if pi >= 0 else None,
             max_pooled_pages=b.summary_width[stream] if pi >= 0 else 0, pool=m.pool if pi >= 0 else 0,
             window=m.window if windowed else 0, keep_first=m.keep_first if windowed else 0, scale=m.scale, softcap=m.softcap,
-            sink=int(m.sink), chunk=m.chunk or 0, kv_shared=int(m.kv_from is not None))
+            sink=int(m.sink), chunk=m.chunk or 0, kv_shared=int(m.kv_from is not None), q_temp=_lib.ptr(lw.get("temp")),
+            dist_amp=_lib.ptr(lw.get("dist_amp")), dist_rate=_lib.ptr(lw.get("dist_rate")))
         st = self._stream()
         self._check(self.L.lp_window_attn_prep(C.byref(d), b.R, _lib.ptr(b.row_seq), _lib.ptr(b.row_pos), st), "lp_window_attn_prep")
         if pi >= 0:
@@ -953,6 +1025,8 @@ class SeqLMEngine:
     def _dense(self, f: DenseFFConfig, lw, h: torch.Tensor, into=None) -> torch.Tensor:
         if f.act == "clamp_glu":
             up = self.linear(h, lw["w_gu"], self.act, _lib.EPI_CLAMP_GLU, f.limit, GLU_SLOPE)
+        elif f.act == "gelu_glu":
+            up = self.linear(h, lw["w_gu"], self.act, _lib.EPI_GELU_GATE)
         elif f.act == "relu2":
             up = self.linear(h, lw["w_up"], self.act, _lib.EPI_RELU2)
         else:
@@ -1117,6 +1191,8 @@ class SeqLMEngine:
             self._check(rc, "lp_add_positions_f32")
         if cfg.norm == "parallel_dyt":
             return self._forward_parallel(b, want, x, hist)
+        if cfg.norm == "post":
+            return self._forward_post(b, want, x)
         pre = cfg.norm == "pre"
         for li, (lc, lw) in enumerate(zip(cfg.layers, self.w.layers)):
             if self.w.add_before[li] is not None:
@@ -1124,20 +1200,22 @@ class SeqLMEngine:
                 self._check(rc, "lp_add_row_f32")
             if lc.token_shift:      # the normed stream in fp32, then shifted towards the previous token's into the operand dtype
                 hn = self.norm(x, lw["norm1"], F32)
-                h = self._empty((b.R, D), self.act)
+                h = self._empty((b.R, D), F32 if lc.input_conv else self.act)
                 state = self.cache.states[self._shift_index[li]]
                 rc = self.L.lp_token_shift_f32(_lib.ptr(hn), hn.stride(0), _lib.ptr(lw["shift"]), b.R, D, _lib.ptr(b.row_seq),
                                                _lib.ptr(b.row_pos), _lib.ptr(b.seq_row0), _lib.ptr(b.seq_slot), _lib.ptr(state),
                                                state.stride(0), _lib.ptr(h), h.stride(0), int(h.dtype == F32), self._stream())
                 self._check(rc, "lp_token_shift_f32")
+                if lc.input_conv:
+                    h = self.convolved(h, li, "conv1", b)
             else:
-                h = self.norm(x, lw["norm1"], self.act)
+                h = self.operand(x, lw["norm1"], li, "conv1", b)
             if pre:        # x <- x + m * mixer(norm(x)): the update is the store of the mixer's output product
                 self._mix(li, lc.mixer, lw, h, b, into=(x, cfg.residual_mult))
             else:
                 self.norm(self._mix(li, lc.mixer, lw, h, b), lw["norm1b"], accum=x)
             if lc.ff is not None:
-                h = self.norm(x, lw["norm2"], self.act)
+                h = self.operand(x, lw["norm2"], li, "conv2", b)
                 if pre and isinstance(lc.ff, DenseFFConfig):
                     self._dense(lc.ff, lw, h, into=(x, cfg.residual_mult))
                 elif pre:
@@ -1157,6 +1235,39 @@ class SeqLMEngine:
         rows = x if isinstance(want, str) else x.index_select(0, want.long())
         hn = self.dyt(rows, self.w.final_gain)[0] if self.cfg.norm == "parallel_dyt" else self.norm(rows, self.w.final_gain, self.act)
         return self.linear(hn, self.w.head, F32)
+
+    def _forward_post(self, b: _Batch, want, x: torch.Tensor) -> Optional[torch.Tensor]:
+        """Layers whose norm follows the sum: x <- norm(post_alpha x + sublayer(x)).  One kernel closes a sublayer and writes the operand
+        of the next one on the way: the new x in the operand dtype, in one-token steps with the next sublayer's convolution applied;
+        in prompts that convolution is a kernel of its own (its rows look at their neighbours)."""
+        cfg, R, D = self.cfg, b.R, self.cfg.width
+        subs = [(li, which) for li, lc in enumerate(cfg.layers) for which in (("conv1", "conv2") if lc.ff is not None else ("conv1",))]
+        h = None
+        for k, (li, which) in enumerate(subs):
+            lc, lw = cfg.layers[li], self.w.layers[li]
+            if h is None:      # the first sublayer of the stack, and convolutions that did not ride on the norm before them
+                h = self.convolved(x, li, which, b) if lc.input_conv else x if self.act == F32 else x.to(self.act)
+            if which == "conv1":
+                y = self._mix(li, lc.mixer, lw, h, b)
+            else:
+                y = self._dense(lc.ff, lw, h) if isinstance(lc.ff, DenseFFConfig) else self._moe(lc.ff, lw, h)
+            nli, nwhich = subs[k + 1] if k + 1 < len(subs) else (None, None)
+            taps = cfg.layers[nli].input_conv if nli is not None else 0
+            ride = nli is not None and (b.decode if taps else self.act != F32)
+            h = self._empty((R, D), self.act) if ride else None
+            state = self._conv_state(nli, nwhich) if ride else None
+            conv_w = self.w.layers[nli][nwhich] if ride and taps else None
+            rc = self.L.lp_post_norm_f32(_lib.ptr(x), x.stride(0), _lib.ptr(y), y.stride(0), float(cfg.post_alpha), R, D,
+                                         _lib.ptr(lw["norm1" if which == "conv1" else "norm2"]), cfg.eps, _lib.ptr(h),
+                                         h.stride(0) if h is not None else 0, int(self.act == F32), _lib.ptr(conv_w), taps,
+                                         _lib.ptr(b.row_pos), _lib.ptr(b.seq_slot), _lib.ptr(state),
+                                         state.stride(0) if state is not None else 0, self._stream())
+            self._check(rc, "lp_post_norm_f32")
+            if self.tap is not None and nli != li:
+                self.tap(li, x)
+        if want is None:
+            return None
+        return self._head(x, want)
 
     def _forward_parallel(self, b: _Batch, want, x0: torch.Tensor, hist: Optional[torch.Tensor]) -> Optional[torch.Tensor]:
         """Layers whose two sublayers read the SAME stream through two Dynamic-Tanh norms: X' = x + m (gate1 * mixer(norm1 x) + gate2 *
