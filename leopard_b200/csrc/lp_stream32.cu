@@ -387,8 +387,9 @@ struct ConvLaunch {
 template <typename OT, int V, int K>
 static void launch_conv(const ConvLaunch& a, cudaStream_t stream) {
   const int subs = (a.longest + CONV_TILE - 1) / CONV_TILE;
-  const dim3 grid(a.n_chunks * subs, (a.D / V + CONV_THREADS - 1) / CONV_THREADS);
-  causal_conv_kernel<OT, V, K><<<grid, CONV_THREADS, 0, stream>>>(a.h, a.ldh, a.w, a.D, a.chunk_seq, a.chunk_row0, a.chunk_len, subs, CONV_TILE,
+  const int cols = a.D / V, threads = cols >= CONV_THREADS ? CONV_THREADS : (cols + 31) / 32 * 32;
+  const dim3 grid(a.n_chunks * subs, (cols + threads - 1) / threads);
+  causal_conv_kernel<OT, V, K><<<grid, threads, 0, stream>>>(a.h, a.ldh, a.w, a.D, a.chunk_seq, a.chunk_row0, a.chunk_len, subs, CONV_TILE,
                                                                  a.row_pos, a.seq_row0, a.seq_slot, a.state, a.slot_stride,
                                                                  reinterpret_cast<OT*>(a.out), a.ldo);
 }

@@ -17,6 +17,10 @@
 #include <memory>
 #include <thread>
 #include <vector>
+#ifdef EMU_FIBERS
+#include <setjmp.h>
+#include <ucontext.h>
+#endif
 
 #define __global__
 #define __device__
@@ -76,6 +80,119 @@ using std::min;
 using std::max;
 
 // ---- block / warp synchronisation ----------------------------------------------------------------------------------------
+#ifdef EMU_FIBERS
+// One OS thread, one fiber per CUDA thread: a block's fibers take turns, giving way inside every barrier.  Much faster than an OS thread per
+// CUDA thread where nothing spins on memory (no mbarriers); a barrier that can never fill is reported instead of hanging.
+namespace emu {
+struct Fiber {
+  ucontext_t start;
+  jmp_buf at;
+  bool entered = false, done = false;
+};
+struct Scheduler {
+  jmp_buf home;
+  std::vector<Fiber> fibers;
+  unsigned current = 0;
+  unsigned long long progress = 0;      // barriers filled and fibers finished
+};
+inline Scheduler* g_sched = nullptr;
+inline void give_way() {
+  Fiber& f = g_sched->fibers[g_sched->current];
+  if (_setjmp(f.at) == 0) _longjmp(g_sched->home, 1);
+}
+struct Barrier {
+  int expected = 0, arrived = 0;
+  unsigned turn = 0;
+  explicit Barrier(int n) : expected(n) {}
+  void fill() {
+    arrived = 0;
+    ++turn;
+    ++g_sched->progress;
+  }
+  void arrive_and_wait() {
+    const unsigned mine = turn;
+    if (++arrived >= expected) fill();
+    else
+      while (turn == mine) give_way();
+  }
+  void arrive_and_drop() {
+    if (--expected > 0 && arrived >= expected) fill();
+  }
+};
+struct BlockCtx {
+  std::unique_ptr<Barrier> block_bar;
+  std::vector<std::unique_ptr<Barrier>> warp_bar;
+  std::vector<float> warp_buf;   // [warps][32]
+  std::map<std::pair<unsigned, unsigned>, std::unique_ptr<Barrier>> sub_bar;
+  Barrier& group(unsigned warp, unsigned mask) {
+    if (mask == 0xffffffffu) return *warp_bar[warp];
+    auto& b = sub_bar[{warp, mask}];
+    if (!b) b = std::make_unique<Barrier>(__builtin_popcount(mask));
+    return *b;
+  }
+};
+inline BlockCtx* t_ctx = nullptr;
+inline std::function<void()>* g_body = nullptr;
+inline void fiber_main() {
+  (*g_body)();
+  t_ctx->block_bar->arrive_and_drop();      // a thread that has returned no longer takes part in __syncthreads
+  g_sched->fibers[g_sched->current].done = true;
+  ++g_sched->progress;
+  _longjmp(g_sched->home, 1);
+}
+template <typename F>
+void launch(dim3 grid, dim3 block, F&& body) {
+  constexpr size_t STACK = 128 * 1024;
+  const unsigned n = block.x * block.y * block.z, n_warps = (n + 31) / 32;
+  const unsigned long long n_blocks = (unsigned long long)grid.x * grid.y * grid.z;
+  static std::vector<std::unique_ptr<char[]>> stacks;
+  while (stacks.size() < n) stacks.emplace_back(new char[STACK]);
+  Scheduler sched;
+  sched.fibers.resize(n);
+  std::function<void()> fn = body;
+  g_sched = &sched;
+  g_body = &fn;
+  blockDim = block;
+  gridDim = grid;
+  for (unsigned long long b = 0; b < n_blocks; ++b) {
+    BlockCtx ctx;
+    ctx.block_bar = std::make_unique<Barrier>((int)n);
+    for (unsigned w = 0; w < n_warps; ++w) ctx.warp_bar.push_back(std::make_unique<Barrier>((int)std::min(32u, n - w * 32)));
+    ctx.warp_buf.assign(n_warps * 32, 0.f);
+    t_ctx = &ctx;
+    blockIdx = {(unsigned)(b % grid.x), (unsigned)((b / grid.x) % grid.y), (unsigned)(b / ((unsigned long long)grid.x * grid.y))};
+    for (auto& f : sched.fibers) f.entered = f.done = false;
+    volatile unsigned left = n;
+    while (left) {
+      const unsigned long long before = sched.progress;
+      for (volatile unsigned t = 0; t < n; t = t + 1) {
+        Fiber& f = sched.fibers[t];
+        if (f.done) continue;
+        sched.current = t;
+        threadIdx = {t % block.x, (t / block.x) % block.y, t / (block.x * block.y)};
+        if (_setjmp(sched.home) == 0) {
+          if (f.entered) _longjmp(f.at, 1);
+          f.entered = true;
+          getcontext(&f.start);
+          f.start.uc_stack.ss_sp = stacks[t].get();
+          f.start.uc_stack.ss_size = STACK;
+          f.start.uc_link = nullptr;
+          makecontext(&f.start, fiber_main, 0);
+          setcontext(&f.start);
+        }
+        if (sched.fibers[t].done) left = left - 1;
+      }
+      if (left && sched.progress == before) {
+        std::fprintf(stderr, "emu: every remaining thread of a block waits at a barrier that cannot fill\n");
+        std::abort();
+      }
+    }
+  }
+  t_ctx = nullptr;
+  g_sched = nullptr;
+}
+}  // namespace emu
+#else
 namespace emu {
 struct BlockCtx {
   std::unique_ptr<std::barrier<>> block_bar;
@@ -131,6 +248,9 @@ void launch(dim3 grid, dim3 block, F&& body) {
     });
   for (auto& th : ts) th.join();
 }
+}  // namespace emu
+#endif
+namespace emu {
 inline unsigned linear_tid() { return threadIdx.x + blockDim.x * (threadIdx.y + blockDim.y * threadIdx.z); }
 }  // namespace emu
 
@@ -138,7 +258,7 @@ inline void __syncthreads() { emu::t_ctx->block_bar->arrive_and_wait(); }
 inline float __shfl_xor_sync(unsigned mask, float v, int lane_mask) {
   const unsigned t = emu::linear_tid(), w = t >> 5, l = t & 31;
   float* buf = emu::t_ctx->warp_buf.data() + w * 32;
-  std::barrier<>& bar = emu::t_ctx->group(w, mask);
+  auto& bar = emu::t_ctx->group(w, mask);
   buf[l] = v;
   bar.arrive_and_wait();
   const float r = buf[l ^ (unsigned)lane_mask];

@@ -3,6 +3,7 @@ AND their host entry points) for the CPU emulator: includes dropped, dynamic sha
 rewritten (launch_rewrite.py), runtime names from host_emu.h.  The result exports the same C symbols as the native library."""
 import subprocess
 import sys
+from concurrent.futures import ThreadPoolExecutor
 from pathlib import Path
 
 ROOT = Path(__file__).resolve().parents[2]
@@ -32,9 +33,16 @@ def build_emulated(out: Path) -> Path:
         '#include "host_emu.h"\nextern "C" {\nconst char* lp_last_error(void) { return lp::g_emu_err; }\n'
         'long long lp_launch_count(void) { return 0; }\nint lp_abi_version(void) { return 3; }\n}\n')
     lib = out / "libstream32_emu.so"
-    r = subprocess.run(["g++", "-std=c++20", "-O2", "-pthread", "-shared", "-fPIC", "-ffp-contract=off", "-fno-strict-aliasing", "-I", str(out),
-                        "-I", str(ROOT / "tests/emu"), "-I", str(ROOT / "include"), *units, str(out / "common_emu.cpp"), "-o", str(lib)],
-                       capture_output=True, text=True)
-    if r.returncode != 0:
-        raise RuntimeError(r.stderr[-6000:])
+    flags = ["-std=c++20", "-O2", "-pthread", "-fPIC", "-ffp-contract=off", "-fno-strict-aliasing", "-DEMU_FIBERS", "-U_FORTIFY_SOURCE",
+             "-I", str(out), "-I", str(ROOT / "tests/emu"), "-I", str(ROOT / "include")]
+
+    def run(cmd):
+        r = subprocess.run(cmd, capture_output=True, text=True)
+        if r.returncode != 0:
+            raise RuntimeError(r.stderr[-6000:])
+
+    units.append(str(out / "common_emu.cpp"))
+    with ThreadPoolExecutor(max_workers=8) as ex:
+        list(ex.map(lambda u: run(["g++", *flags, "-c", u, "-o", u.replace(".cpp", ".o")]), units))
+    run(["g++", "-shared", "-pthread", *[u.replace(".cpp", ".o") for u in units], "-o", str(lib)])
     return lib
