@@ -216,12 +216,12 @@ def test_attention_over_everything_keeps_every_page(backend):
 @pytest.mark.gpu
 def test_far_keys_and_edges_among_hundreds():
     """windows of hundreds of keys and causal attention over everything (several key tiles, many pages), sharp softmaxes: the oracle
-    with a window one token off, a distance one token off and a changed first token is told apart; portions start at every kind of
+    with a window one token off and a changed first token is told apart; portions start at every kind of
     offset and the end is decoded"""
-    layers = [latent_layer(heads=4, dim=8, rot_dim=8, vdim=8, q_rank=12, kv_rank=16, window=150, scale=1.5),
-              attention_layer(heads=8, kv_heads=2, dim=16, vdim=8, scale=2.0),
-              latent_layer(heads=2, dim=8, rot_dim=8, vdim=8, q_rank=12, kv_rank=16, window=131, scale=1.5, kv_from=0)]
-    cfg = model(layers, width=24, taps=4)
+    layers = [latent_layer(heads=16, dim=8, rot_dim=8, vdim=8, q_rank=12, kv_rank=16, window=150, scale=0.7),
+              attention_layer(heads=8, kv_heads=2, dim=16, vdim=8, scale=1.0),
+              latent_layer(heads=12, dim=8, rot_dim=8, vdim=8, q_rank=12, kv_rank=16, window=131, scale=0.7, kv_from=0)]
+    cfg = model(layers, width=24, taps=4, alpha=1.5)
     w = O.random_weights(cfg, seed=31)
     w["l1.mix.r1"] = w["l1.mix.r1"] * 0.2
     toks = _tokens(330, cfg["vocab"], seed=32)
@@ -229,9 +229,9 @@ def test_far_keys_and_edges_among_hundreds():
     for li in (0, 2):
         for delta in (-1, 1):
             off = _rows(O.forward(_one_off(cfg, delta, li), w, toks), want)
-            assert int((off[150:] > 200 * TOL["float32"]).sum()) >= 40
+            assert int((off[150:] > 200 * TOL["float32"]).sum()) >= 15
     first = O.forward(cfg, w, [(toks[0] + 1) % cfg["vocab"]] + toks[1:])      # the causal layer remembers token 0
-    assert int((_rows(first[-100:], want[-100:]) > 20 * TOL["float32"]).sum()) >= 20
+    assert int((_rows(first[-100:], want[-100:]) > 20 * TOL["float32"]).sum()) >= 50
     eng = make_engine(cfg, w, ("cuda", None), max_tokens=400, page_size=16)
     got, at = [], 0
     for n in (129, 2, 67, 101, 3):
