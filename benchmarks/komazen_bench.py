@@ -109,13 +109,13 @@ def bench_komazen(name, s, dev, steps, warmup, peaks, prompt):
     def per_s(k, amount, unit):
         return round(amount / (k["ms"] * 1e-3) / unit, 2) if k and k["ms"] > 0 else None
     r = {}
-    for key, flops in (("lp_gemm_bf16", flops_gemm), ("lp_window_attn_tiles", attn_flops), ("lp_latent_attend", lat_flops)):
+    for key, flops in (("lp_gemm_bf16", flops_gemm), ("lp_window_attn_tiles", attn_flops), ("lp_latent_attend_tiles", lat_flops)):
         r[key + "_tflops"] = per_s(kp.get(key), flops, 1e12)
     heads_key = "lp_linear_heads" if "lp_linear_heads" in kp else "lp_linear"
     r["per_head_products_tflops"] = per_s(kp.get(heads_key), head_flops, 1e12)
     if r["lp_gemm_bf16_tflops"]:
         r["lp_gemm_bf16_of_bf16_peak"] = round(r["lp_gemm_bf16_tflops"] / peaks["bf16_burst"], 3)
-    for k in ("lp_window_attn_tiles", "lp_latent_attend", "per_head_products"):
+    for k in ("lp_window_attn_tiles", "lp_latent_attend_tiles", "per_head_products"):
         if r[k + "_tflops"]:
             r[k + "_of_fp32_fma_peak"] = round(r[k + "_tflops"] / FP32_FMA_TFLOPS, 3)
     for k, nbytes in elem_bytes.items():

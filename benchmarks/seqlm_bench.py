@@ -178,7 +178,7 @@ def bench_size(name, s, dev, steps, warmup, peaks, prompt):
     out["prefill_rates"] = {
         "lp_gemm_bf16_tflops": rate("lp_gemm_bf16", flops_gemm), "of_bf16_peak": None,
         "lp_retention_prefill_tflops": rate("lp_retention_prefill", ret_flops),
-        "lp_latent_attend_tflops": rate("lp_latent_attend", lat_flops),
+        "lp_latent_attend_tflops": rate("lp_latent_attend_tiles", lat_flops),
         "lp_linear_grouped_tflops": rate("lp_linear_grouped", moe_flops)}
     if out["prefill_rates"]["lp_gemm_bf16_tflops"]:
         out["prefill_rates"]["of_bf16_peak"] = round(out["prefill_rates"]["lp_gemm_bf16_tflops"] / peaks["bf16_burst"], 3)

@@ -688,6 +688,11 @@ int lp_latent_prep(const lp_latent_desc* desc, int R, const int* row_seq, const 
 /* q_abs fp32 [rows, heads * kv_rank] = per-head W_uk^T q_unrotated; out [rows, heads * kv_rank] = softmax-weighted sum of cached c */
 int lp_latent_attend(const lp_latent_desc* desc, int R, const int* row_seq, const int* row_pos, const float* q_abs, long long ldqa,
                      void* out, long long ldo, int out_fp32, void* stream);
+/* the same result for the rows of prompts, per tile of (row, head) pairs of one request that share the keys they read (chunk tables as
+ * for lp_retention_prefill).  Few rows, and sizes the tiles do not take, go to lp_latent_attend. */
+int lp_latent_attend_tiles(const lp_latent_desc* desc, int R, const int* row_seq, const int* row_pos, int n_chunks, const int* chunk_seq,
+                           const int* chunk_row0, const int* chunk_len, const float* q_abs, long long ldqa, void* out, long long ldo,
+                           int out_fp32, void* stream);
 
 /* Grouped-query attention over a paged cache of rows [keys (kv_heads x dim) | values (kv_heads x vdim)] fp32, with the visibility
  * rules and score options of sliding-window designs as parameters (csrc/lp_winattn.cu).  Query at position i of a request sees

@@ -256,6 +256,7 @@ _SIGS = {
     "lp_retention_decode": (_i, [C.POINTER(RetentionDesc), _i, _vp, _vp, _vp, _vp]),
     "lp_latent_prep": (_i, [C.POINTER(LatentDesc), _i, _vp, _vp, _vp]),
     "lp_latent_attend": (_i, [C.POINTER(LatentDesc), _i, _vp, _vp, _vp, _ll, _vp, _ll, _i, _vp]),
+    "lp_latent_attend_tiles": (_i, [C.POINTER(LatentDesc), _i, _vp, _vp, _i, _vp, _vp, _vp, _vp, _ll, _vp, _ll, _i, _vp]),
     "lp_moe_route": (_i, [_vp, _ll, _i, _i, _i, _vp, _ll, _i, _vp, _i, _i, _i, _vp, _vp, _vp, _vp, _vp]),
     "lp_moe_max_tiles": (_i, [_i, _i, _i]),
     "lp_moe_align": (_i, [_vp, _i, _i, _i, _i, _i, _vp, _vp, _vp, _vp]),
@@ -309,7 +310,7 @@ STREAM32_SYMBOLS = ("lp_last_error", "lp_abi_version", "lp_launch_count", "lp_li
                     "lp_mingru_prefill", "lp_mingru_decode", "lp_window_attn_talk", "lp_window_attn_talk_tiles", "lp_mlstm_workspace_bytes", "lp_mlstm",
                     "lp_add_positions_f32", "lp_add_row_f32", "lp_token_shift_f32", "lp_moe_route_softmax", "lp_glu_scaled_f32", "lp_dyt_f32",
                     "lp_rmsnorm_gated_f32", "lp_gated_axpy_f32", "lp_depth_average_f32", "lp_moe_route_sigmoid", "lp_moe_sorted_weights",
-                    "lp_causal_conv_max_taps", "lp_causal_conv_f32", "lp_post_norm_f32")
+                    "lp_causal_conv_max_taps", "lp_causal_conv_f32", "lp_post_norm_f32", "lp_latent_attend_tiles")
 STREAM32_OPTIONAL = ("lp_gemm_bf16",)      # present in the native libraries, absent from the CPU-emulated build
 _stream32 = None
 

@@ -23,6 +23,8 @@
 //       lp_latent_prep   RMS-norms the latent (vector gain), rotates the shared key part and writes both to the request's pages;
 //                        rotates the query's rotated part in place (without latents of its own: only that).
 //       lp_latent_attend one CTA per (row, head), its warps split the visible keys: online softmax in fp32, merged at the end.
+//       lp_latent_attend_tiles  prompts: tiles of (row, head) pairs share the keys they read.
+#include <cuda_pipeline.h>
 #include "lp_host.h"
 #include "../../include/leopard_b200.h"
 
@@ -605,6 +607,181 @@ latent_attend_rows_kernel(LatArgs a, int R, const int* __restrict__ row_seq, con
   }
 }
 
+// Prompts, tiled: a CTA takes LT_X = 64 (row, head) pairs of one request's chunk — all heads read the same latents, so the pairs share
+// every key — and walks the union of what its rows see, LT_K = 16 keys at a time; every pair is masked by its row's own rule.  Both halves
+// are register-tiled fp32 products fed from shared memory: scores 4 pairs x 2 keys a thread with two lanes splitting the channels, sums
+// 8 pairs x (4 NC) latent channels a thread (NC = ceil(kv_rank / 128)).  The next tile of keys is copied in (cp.async) while this one is
+// worked on.  Rows in shared memory are LD floats apart, LD = 8 mod 32, so that the 8 sixteen-byte pieces a score load of a warp touches
+// lie in different banks; the padding is zero and takes part in the sums.
+constexpr int LT_X = 64, LT_K = 16, LT_THREADS = 256, LT_PS = LT_X + 4, LT_MAX_NC = 4;
+static int lt_ld(int width) { return (width + 23) / 32 * 32 + 8; }      // the smallest number >= width that is 8 mod 32
+static size_t lt_smem_floats(int width) { return (size_t)(LT_X + 2 * LT_K) * lt_ld(width) + LT_K * LT_PS + LT_X; }
+
+template <int NC>
+__global__ void __launch_bounds__(LT_THREADS)
+latent_attend_tile_kernel(LatArgs a, int ld, int n_chunks, const int* __restrict__ chunk_seq, const int* __restrict__ chunk_row0,
+                          const int* __restrict__ chunk_len, int tiles_per_chunk, const int* __restrict__ row_pos,
+                          const float* __restrict__ q_abs, long long ldqa, void* __restrict__ out, long long ldo, int out_fp32) {
+  extern __shared__ float dyn_smem[];
+  const int ck = blockIdx.x / tiles_per_chunk, v0 = (blockIdx.x % tiles_per_chunk) * LT_X;
+  const int H = a.heads, C = a.kv_rank, width = a.kv_rank + a.rot_dim;
+  if (ck >= n_chunks || v0 >= chunk_len[ck] * H) return;
+  const int nv = min(LT_X, chunk_len[ck] * H - v0);      // pairs of this tile: pair x is row (v0 + x) / H, head (v0 + x) % H
+  const int r0 = chunk_row0[ck], seq = chunk_seq[ck];
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  float* q_s = dyn_smem;                        // [LT_X][ld]
+  float* k_s = q_s + LT_X * ld;                 // [2][LT_K][ld]
+  float* p_s = k_s + 2 * LT_K * ld;             // [LT_K][LT_PS] scores, then weights
+  float* corr_s = p_s + LT_K * LT_PS;           // [LT_X] what the running sums are multiplied by
+  for (int i = tid; i < LT_X * ld; i += LT_THREADS) {
+    const int x = i / ld, d = i % ld;
+    float v = 0.f;
+    if (x < nv && d < width) {
+      const long long r = r0 + (v0 + x) / H;
+      const int h = (v0 + x) % H;
+      v = d < C ? q_abs[r * ldqa + (long long)h * C + d] : a.q[r * a.ldq + (long long)h * (a.dim + a.rot_dim) + a.dim + (d - C)];
+    }
+    q_s[i] = v;
+  }
+  for (int i = tid; i < 2 * LT_K * ld; i += LT_THREADS) k_s[i] = 0.f;      // padding, and keys past the end (their weight is zero)
+  const int pos_first = row_pos[r0 + v0 / H], pos_last = row_pos[r0 + (v0 + nv - 1) / H];
+  const int lo = (a.window > 0 && pos_first - a.window + 1 > 0) ? pos_first - a.window + 1 : 0;
+  const int n_keys = pos_last - lo + 1, pieces = width >> 2, steps = (pieces + 1) & ~1;
+  auto load = [&](int t0, float* dst) {
+    for (int j = warp; j < LT_K; j += LT_THREADS / 32) {
+      if (t0 + j >= n_keys) break;
+      const float* src = lat_cache_row(a, seq, lo + t0 + j);
+      for (int p = lane; p < pieces; p += 32) __pipeline_memcpy_async(dst + j * ld + 4 * p, src + 4 * p, 16);
+    }
+    __pipeline_commit();
+  };
+  // the pair whose softmax this thread keeps, together with the three lanes beside it
+  const int sx = tid >> 2, part = tid & 3;
+  const int my_pos = sx < nv ? row_pos[r0 + (v0 + sx) / H] : -1;
+  const int my_lo = sx < nv ? ((a.window > 0 && my_pos - a.window + 1 > 0) ? my_pos - a.window + 1 : 0) : 0x7fffffff;
+  const int my_h = (v0 + sx) % H;
+  float mx = a.sink != nullptr ? a.sink[my_h] : -INFINITY, den = a.sink != nullptr ? 1.f : 0.f;
+  const int sl = lane & 1, x_at = (warp & 3) * 16 + ((lane >> 1) & 3), k_at = (warp >> 2) * 8 + (lane >> 3);
+  float acc[8][4 * NC];
+#pragma unroll
+  for (int x = 0; x < 8; ++x)
+#pragma unroll
+    for (int i = 0; i < 4 * NC; ++i) acc[x][i] = 0.f;
+  __syncthreads();
+  load(0, k_s);
+  for (int t0 = 0; t0 < n_keys; t0 += LT_K) {
+    const float* kt = k_s + ((t0 / LT_K) & 1) * LT_K * ld;
+    __pipeline_wait_prior(0);
+    __syncthreads();      // the tile is here for everyone, and nobody reads the other buffer or the weights any more
+    if (t0 + LT_K < n_keys) load(t0 + LT_K, k_s + ((t0 / LT_K + 1) & 1) * LT_K * ld);
+    {
+      float s[4][2];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) s[i][0] = s[i][1] = 0.f;
+      const float* qp = q_s + x_at * ld + 4 * sl;
+      const float* kp = kt + k_at * ld + 4 * sl;
+#pragma unroll 4
+      for (int g = 0; g < steps; g += 2) {
+        float4 k4[2];
+#pragma unroll
+        for (int j = 0; j < 2; ++j) k4[j] = *reinterpret_cast<const float4*>(kp + 4 * j * ld + 4 * g);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const float4 q4 = *reinterpret_cast<const float4*>(qp + 4 * i * ld + 4 * g);
+#pragma unroll
+          for (int j = 0; j < 2; ++j) {
+            s[i][j] = fmaf(q4.x, k4[j].x, s[i][j]);
+            s[i][j] = fmaf(q4.y, k4[j].y, s[i][j]);
+            s[i][j] = fmaf(q4.z, k4[j].z, s[i][j]);
+            s[i][j] = fmaf(q4.w, k4[j].w, s[i][j]);
+          }
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+#pragma unroll
+        for (int j = 0; j < 2; ++j) s[i][j] += __shfl_xor_sync(0xffffffffu, s[i][j], 1);
+        p_s[(k_at + 4 * sl) * LT_PS + x_at + 4 * i] = sl ? s[i][1] : s[i][0];
+      }
+    }
+    __syncthreads();
+    {
+      float v[LT_K / 4], top = -INFINITY;
+#pragma unroll
+      for (int j = 0; j < LT_K / 4; ++j) {
+        const int key = part * (LT_K / 4) + j, at = lo + t0 + key;
+        v[j] = (at >= my_lo && at <= my_pos) ? p_s[key * LT_PS + sx] * a.scale : -INFINITY;
+        top = fmaxf(top, v[j]);
+      }
+      top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, 1));
+      top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, 2));
+      const float mn = fmaxf(mx, top), ref = mn == -INFINITY ? 0.f : mn;      // -inf: this pair has seen nothing yet
+      const float corr = expf(mx - ref);
+      float sum = 0.f;
+#pragma unroll
+      for (int j = 0; j < LT_K / 4; ++j) {
+        const float p = expf(v[j] - ref);
+        p_s[(part * (LT_K / 4) + j) * LT_PS + sx] = p;
+        sum += p;
+      }
+      sum += __shfl_xor_sync(0xffffffffu, sum, 1);
+      sum += __shfl_xor_sync(0xffffffffu, sum, 2);
+      den = fmaf(den, corr, sum);
+      mx = mn;
+      if (part == 0) corr_s[sx] = corr;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int x = 0; x < 8; ++x) {
+      const float c = corr_s[warp * 8 + x];      // the same for the whole warp
+      if (c != 1.f) {
+#pragma unroll
+        for (int i = 0; i < 4 * NC; ++i) acc[x][i] *= c;
+      }
+    }
+    const float* wp = p_s + warp * 8;
+    const float* cp = kt + 4 * lane;
+#pragma unroll 2
+    for (int jj = 0; jj < LT_K; ++jj) {
+      const float4 w0 = *reinterpret_cast<const float4*>(wp + jj * LT_PS), w1 = *reinterpret_cast<const float4*>(wp + jj * LT_PS + 4);
+      const float w[8] = {w0.x, w0.y, w0.z, w0.w, w1.x, w1.y, w1.z, w1.w};
+#pragma unroll
+      for (int i = 0; i < NC; ++i) {
+        if (4 * lane + 128 * i < C) {
+          const float4 c4 = *reinterpret_cast<const float4*>(cp + jj * ld + 128 * i);
+#pragma unroll
+          for (int x = 0; x < 8; ++x) {
+            acc[x][4 * i] = fmaf(w[x], c4.x, acc[x][4 * i]);
+            acc[x][4 * i + 1] = fmaf(w[x], c4.y, acc[x][4 * i + 1]);
+            acc[x][4 * i + 2] = fmaf(w[x], c4.z, acc[x][4 * i + 2]);
+            acc[x][4 * i + 3] = fmaf(w[x], c4.w, acc[x][4 * i + 3]);
+          }
+        }
+      }
+    }
+  }
+  __syncthreads();
+  if (part == 0) corr_s[sx] = sx < nv ? lat_gate(a, r0 + (v0 + sx) / H, my_h) / den : 0.f;
+  __syncthreads();
+#pragma unroll
+  for (int x = 0; x < 8; ++x) {
+    const int v = v0 + warp * 8 + x;
+    if (warp * 8 + x >= nv) break;
+    const float f = corr_s[warp * 8 + x];
+    const long long at = (long long)(r0 + v / H) * ldo + (long long)(v % H) * C + 4 * lane;
+#pragma unroll
+    for (int i = 0; i < NC; ++i) {
+      if (4 * lane + 128 * i < C) {
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+          if (out_fp32) reinterpret_cast<float*>(out)[at + 128 * i + k] = acc[x][4 * i + k] * f;
+          else reinterpret_cast<bf16*>(out)[at + 128 * i + k] = __float2bfloat16(acc[x][4 * i + k] * f);
+        }
+      }
+    }
+  }
+}
+
 // raise a kernel's dynamic shared-memory limit only when a launch needs more than any launch before it (no runtime call on the
 // steady path, so the steady path can be captured into a CUDA graph)
 template <typename K>
@@ -749,4 +926,41 @@ extern "C" int lp_latent_attend(const lp_latent_desc* d, int R, const int* row_s
   note_launch();
   LP_CHECK_CUDA(cudaGetLastError());
   return 0;
+}
+
+template <int NC>
+static int launch_latent_tiles(const LatArgs& a, int R, int n_chunks, const int* chunk_seq, const int* chunk_row0, const int* chunk_len,
+                               const int* row_pos, const float* q_abs, long long ldqa, void* out, long long ldo, int out_fp32, cudaStream_t stream) {
+  static size_t have = 48 * 1024;
+  const int width = a.kv_rank + a.rot_dim;
+  const size_t smem = lt_smem_floats(width) * sizeof(float);
+  LP_CHECK_CUDA(ensure_smem(latent_attend_tile_kernel<NC>, smem, have));
+  const int longest = R < LP_RETENTION_CHUNK ? R : LP_RETENTION_CHUNK;      // no chunk has more rows than the step or the chunk size
+  const int tiles = (longest * a.heads + LT_X - 1) / LT_X;
+  latent_attend_tile_kernel<NC><<<n_chunks * tiles, LT_THREADS, smem, stream>>>(a, lt_ld(width), n_chunks, chunk_seq, chunk_row0, chunk_len, tiles,
+                                                                                row_pos, q_abs, ldqa, out, ldo, out_fp32);
+  note_launch();
+  LP_CHECK_CUDA(cudaGetLastError());
+  return 0;
+}
+
+extern "C" int lp_latent_attend_tiles(const lp_latent_desc* d, int R, const int* row_seq, const int* row_pos, int n_chunks,
+                                      const int* chunk_seq, const int* chunk_row0, const int* chunk_len, const float* q_abs, long long ldqa,
+                                      void* out, long long ldo, int out_fp32, void* stream_) {
+  cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
+  LatArgs a;
+  if (int rc = fill_lat(a, d)) return rc;
+  LP_REQUIRE(q_abs != nullptr && out != nullptr && row_seq != nullptr && row_pos != nullptr && chunk_seq != nullptr && chunk_row0 != nullptr &&
+                 chunk_len != nullptr,
+             "lp_latent_attend_tiles: null operand");
+  if (R <= 0 || n_chunks <= 0) return 0;
+  const int width = d->kv_rank + d->rot_dim, nc = (d->kv_rank + 127) / 128;
+  // 16-byte pieces of the cache rows, all of a pair's sums in registers, both operands in shared memory; few rows are split over keys
+  if (R <= LP_LATENT_SPLIT_ROWS || d->kv_rank % 4 || d->rot_dim % 4 || nc > LT_MAX_NC || lt_smem_floats(width) * sizeof(float) > 227 * 1024 ||
+      (reinterpret_cast<uintptr_t>(d->cache) & 15))
+    return lp_latent_attend(d, R, row_seq, row_pos, q_abs, ldqa, out, ldo, out_fp32, stream_);
+  if (nc == 1) return launch_latent_tiles<1>(a, R, n_chunks, chunk_seq, chunk_row0, chunk_len, row_pos, q_abs, ldqa, out, ldo, out_fp32, stream);
+  if (nc == 2) return launch_latent_tiles<2>(a, R, n_chunks, chunk_seq, chunk_row0, chunk_len, row_pos, q_abs, ldqa, out, ldo, out_fp32, stream);
+  if (nc == 3) return launch_latent_tiles<3>(a, R, n_chunks, chunk_seq, chunk_row0, chunk_len, row_pos, q_abs, ldqa, out, ldo, out_fp32, stream);
+  return launch_latent_tiles<4>(a, R, n_chunks, chunk_seq, chunk_row0, chunk_len, row_pos, q_abs, ldqa, out, ldo, out_fp32, stream);
 }

@@ -895,8 +895,13 @@ class SeqLMEngine:
         q_abs = self._empty((b.R, m.heads * m.kv_rank), F32)
         self.linear_heads(q, per, lw["w_ukT"], q_abs, m.kv_rank)
         lat = self._empty((b.R, m.heads * m.kv_rank), self.act)
-        rc = self.L.lp_latent_attend(C.byref(d), b.R, _lib.ptr(b.row_seq), _lib.ptr(b.row_pos), _lib.ptr(q_abs), q_abs.stride(0),
-                                     _lib.ptr(lat), lat.stride(0), int(lat.dtype == F32), self._stream())
+        if b.decode:
+            rc = self.L.lp_latent_attend(C.byref(d), b.R, _lib.ptr(b.row_seq), _lib.ptr(b.row_pos), _lib.ptr(q_abs), q_abs.stride(0),
+                                         _lib.ptr(lat), lat.stride(0), int(lat.dtype == F32), self._stream())
+        else:      # prompts and portions: tiles of (row, head) pairs share the keys they read
+            rc = self.L.lp_latent_attend_tiles(C.byref(d), b.R, _lib.ptr(b.row_seq), _lib.ptr(b.row_pos), b.n_chunks, _lib.ptr(b.chunk_seq),
+                                               _lib.ptr(b.chunk_row0), _lib.ptr(b.chunk_len), _lib.ptr(q_abs), q_abs.stride(0),
+                                               _lib.ptr(lat), lat.stride(0), int(lat.dtype == F32), self._stream())
         self._check(rc, "lp_latent_attend")
         o = self._empty((b.R, m.heads * m.vdim), self.act)
         self.linear_heads(lat, m.kv_rank, lw["w_uv"].view(m.heads, m.vdim, m.kv_rank), o, m.vdim, gate=out_gate)

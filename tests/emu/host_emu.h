@@ -7,6 +7,11 @@
 #include <cstdarg>
 #include <cstdio>
 
+// asynchronous copies into shared memory complete at once
+inline void __pipeline_memcpy_async(void* dst, const void* src, size_t n) { std::memcpy(dst, src, n); }
+inline void __pipeline_commit() {}
+inline void __pipeline_wait_prior(int) {}
+
 typedef void* cudaStream_t;
 typedef int cudaError_t;
 constexpr cudaError_t cudaSuccess = 0;

@@ -17,6 +17,7 @@ def build_emulated(out: Path) -> Path:
     units = []
     for name in SOURCES:
         src = (ROOT / "leopard_b200/csrc" / f"{name}.cu").read_text()
+        src = src.replace('#include <cuda_pipeline.h>\n', "")
         for line in ('#include "lp_host.h"\n', '#include "../../include/leopard_b200.h"\n'):
             assert line in src, (name, line)
             src = src.replace(line, "")

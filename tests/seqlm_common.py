@@ -54,12 +54,17 @@ def plain_model():
                   retention_layer(heads=1, dim=4, vdim=4, rot_dims=4, decay=(0.5,), mlp=dense(ff=9))], width=20, vocab=37, eps=1e-6)
 
 
+_emulated = []      # built once for all test modules that import the fixture
+
+
 @pytest.fixture(scope="session")
 def emu_lib(tmp_path_factory):
-    sys.path.insert(0, str(ROOT / "tests/emu"))
-    from stream32_build import build_emulated
-    from leopard_b200 import _lib
-    return _lib.bind_stream32(C.CDLL(str(build_emulated(tmp_path_factory.mktemp("emu_stream32")))))
+    if not _emulated:
+        sys.path.insert(0, str(ROOT / "tests/emu"))
+        from stream32_build import build_emulated
+        from leopard_b200 import _lib
+        _emulated.append(_lib.bind_stream32(C.CDLL(str(build_emulated(tmp_path_factory.mktemp("emu_stream32"))))))
+    return _emulated[0]
 
 
 @pytest.fixture(params=BACKENDS)

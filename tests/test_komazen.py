@@ -491,3 +491,55 @@ def test_shared_latents_must_fit(emu_lib, layer, key, value):
     bad["layers"][layer]["mixer"][key] = value
     with pytest.raises(ValueError):
         make_engine(bad, O.random_weights(bad, seed=1), ("cpu", emu_lib))
+
+
+@pytest.mark.parametrize("heads, rank, rot, window", [(5, 12, 4, 7), (3, 132, 8, None), (2, 260, 4, 11), (1, 388, 12, 3), (40, 8, 0, 20)])
+def test_latent_tiles_match_the_row_kernel(backend, heads, rank, rot, window):
+    """latent attention by tiles of (row, head) pairs against a plain softmax over the cached rows, with a sink and a head gate: two
+    requests of unequal length (one starts inside its sequence), every number of register columns, heads that straddle tiles"""
+    import ctypes as C
+    from leopard_b200 import _lib
+    from leopard_b200.seqlm import LatentAttentionConfig, LayerConfig, RotaryConfig, SeqLMConfig, SeqLMEngine, _Batch
+    device, lib = backend
+
+    class NoWeights:
+        pass
+    w = NoWeights()
+    w.device = torch.device(device)
+    m = LatentAttentionConfig(heads=heads, dim=4, rot_dim=rot, vdim=4, kv_rank=rank, scale=0.3, rot=RotaryConfig(dims=0, base=1.0), window=window)
+    eng = SeqLMEngine(SeqLMConfig("test", 5, 8, 1e-5, (LayerConfig(m, None),)), w, dtype="float32", max_tokens=96, page_size=4, max_seqs=2, lib=lib)
+    g = torch.Generator().manual_seed(rank)
+    lens, start = {"a": 37, "b": 5}, {"a": 6, "b": 0}
+    total = {k: start[k] + lens[k] for k in lens}
+    c = {k: torch.randn(total[k], rank + rot, generator=g) for k in lens}
+    eng.cache.advance(eng.cache.open("a"), 0)
+    eng.cache.reserve(eng.cache.get("a"), start["a"])
+    eng.cache.get("a").length = start["a"]
+    b = _Batch(eng, [StepEntry(k, [0] * n) for k, n in lens.items()])
+    pool = eng.cache.pools[0]
+    pool.fill_(float("nan"))                                      # rows nobody wrote must not be read
+    for k in lens:
+        pages = eng.cache.get(k).pages
+        for t in range(total[k]):
+            pool[pages[t // 4], t % 4] = c[k][t].to(device)
+    q = torch.randn(b.R, heads * (4 + rot), generator=g).to(device)
+    q_abs = (2.0 * torch.randn(b.R, heads * rank, generator=g)).to(device)
+    sink, gate = torch.randn(heads, generator=g).to(device), torch.randn(b.R, heads, generator=g).to(device)
+    d = _lib.LatentDesc(q=_lib.ptr(q), ldq=q.stride(0), heads=heads, dim=4, rot_dim=rot, kv_rank=rank, eps=1e-5, cache=_lib.ptr(pool), page_size=4,
+                        page_table=_lib.ptr(b.page_table), max_pages=b.max_pages, window=window or 0, scale=0.3, sink=_lib.ptr(sink),
+                        gate=_lib.ptr(gate), ldg=heads)
+    out = torch.full((b.R, heads * rank), float("nan"), device=device)
+    rc = eng.L.lp_latent_attend_tiles(C.byref(d), b.R, _lib.ptr(b.row_seq), _lib.ptr(b.row_pos), b.n_chunks, _lib.ptr(b.chunk_seq),
+                                      _lib.ptr(b.chunk_row0), _lib.ptr(b.chunk_len), _lib.ptr(q_abs), q_abs.stride(0), _lib.ptr(out),
+                                      out.stride(0), 1, eng._stream())
+    eng._check(rc, "lp_latent_attend_tiles")
+    qd, qa, r = q.cpu().double().view(b.R, heads, 4 + rot), q_abs.cpu().double().view(b.R, heads, rank), 0
+    for k in lens:
+        rows = c[k].double()
+        for t in range(start[k], total[k]):
+            lo = max(0, t - window + 1) if window else 0
+            s = (qa[r] @ rows[lo:t + 1, :rank].T + qd[r, :, 4:] @ rows[lo:t + 1, rank:].T) * 0.3
+            p = torch.softmax(torch.cat([s, sink.cpu().double()[:, None]], 1), 1)[:, :-1]
+            want = p @ rows[lo:t + 1, :rank] * torch.sigmoid(gate.cpu().double()[r])[:, None]
+            assert rel_err(out[r].view(heads, rank), want) < TOL["float32"], (k, t)
+            r += 1
