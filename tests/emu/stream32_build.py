@@ -34,7 +34,8 @@ def build_emulated(out: Path) -> Path:
         '#include "host_emu.h"\nextern "C" {\nconst char* lp_last_error(void) { return lp::g_emu_err; }\n'
         'long long lp_launch_count(void) { return 0; }\nint lp_abi_version(void) { return 3; }\n}\n')
     lib = out / "libstream32_emu.so"
-    flags = ["-std=c++20", "-O2", "-pthread", "-fPIC", "-ffp-contract=off", "-fno-strict-aliasing", "-DEMU_FIBERS", "-U_FORTIFY_SOURCE",
+    # no unique symbols: the process may hold other emulated libraries, whose contexts of the same name have the threaded form
+    flags = ["-fno-gnu-unique", "-std=c++20", "-O2", "-pthread", "-fPIC", "-ffp-contract=off", "-fno-strict-aliasing", "-DEMU_FIBERS", "-U_FORTIFY_SOURCE",
              "-I", str(out), "-I", str(ROOT / "tests/emu"), "-I", str(ROOT / "include")]
 
     def run(cmd):

@@ -32,7 +32,9 @@ def test_struct_layouts_match_header(tmp_path):
     pairs = {"lp_vit_dims": _lib.VitDims, "lp_vit_layer_weights": _lib.VitLayerWeights, "lp_vit_weights": _lib.VitWeights,
              "lp_proj_weights": _lib.ProjWeights, "lp_dec_dims": _lib.DecDims, "lp_dec_layer_weights": _lib.DecLayerWeights,
              "lp_dec_weights": _lib.DecWeights, "lp_gemm_desc": _lib.GemmDesc, "lp_tp_desc": _lib.TpDesc,
-             "lp_profile_record": _lib.ProfileRecord}
+             "lp_profile_record": _lib.ProfileRecord, "lp_linear_desc": _lib.LinearDesc, "lp_window_attn_desc": _lib.WindowAttnDesc,
+             "lp_mingru_desc": _lib.MinGRUDesc, "lp_retention_desc": _lib.RetentionDesc, "lp_latent_desc": _lib.LatentDesc,
+             "lp_mlstm_desc": _lib.MLSTMDesc}
     lines = []
     for cname, ct in pairs.items():
         lines.append(f'printf("{cname} %zu\\n", sizeof({cname}));')
