@@ -595,7 +595,8 @@ enum lp_rot_layout { LP_ROT_HALF = 0, LP_ROT_INTERLEAVED = 1 };
  * epi CLAMP_GLU: W = [gate rows; up rows], N' = N / 2, g = min(gate, epi_a), u = clamp(up, -epi_a, epi_a), C = g sigmoid(epi_b g) (u + 1).
  * Before the epilogue an accumulator becomes row_scale[m] * acc + bias[n] (either may be NULL; m is the row of C, for lp_linear_pairs
  * the pair; one problem only).  gate (fp32 [rows of C, ldg], or NULL): the epilogue's result is multiplied by sigmoid(gate[m, n]);
- * problem z of a batch reads gate + z * gate_batch. */
+ * problem z of a batch reads gate + z * gate_batch.  seg_cols > 0: output columns [i seg_cols, (i + 1) seg_cols) multiply the operand at
+ * A + i * a_seg, the columns from (n_segs - 1) seg_cols on that of the last segment (seg_cols a multiple of 8 for M <= 8 rows, else of 64). */
 typedef struct lp_linear_desc {
   const void* A; long long lda; long long a_batch; int a_fp32;
   const void* W; long long ldw; long long w_batch;
@@ -605,6 +606,7 @@ typedef struct lp_linear_desc {
   int c_accum; float c_scale;
   const float* bias; const float* row_scale;
   const float* gate; long long ldg; long long gate_batch;
+  int seg_cols, n_segs; long long a_seg;
 } lp_linear_desc;
 int lp_linear(const lp_linear_desc* desc, void* stream);
 /* row tiles of lp_linear_tile_rows() rows, each multiplied by the weight of group tile_group[tile] (w_batch elements apart; < 0: the
@@ -704,7 +706,7 @@ int lp_latent_attend_tiles(const lp_latent_desc* desc, int R, const int* row_seq
  *     is seen when bP + P - 1 <= i - window); they are the means of the block's cached key and value rows, kept in a second paged
  *     pool `pooled` with one row per block (pooled_table: pages of block rows per request).
  * score = q . k * scale, then softcap * tanh(score / softcap) when softcap > 0, then (dist_amp, dist_rate, both [heads], not with pooled
- * blocks) a distance bias dist_amp[h] * ln(1 + dist_rate[h] * (i - j)) is taken off.  q_temp [heads] multiplies every query head after its
+ * blocks) a distance bias dist_amp[h] * ln(1 + dist_rate[h] * (i - j)), or a linear one, is taken off.  q_temp [heads] multiplies every query head after its
  * norm.  One softmax over everything visible; sink != 0 adds
  * 1 to its denominator (a key of score 0 without a value).  Query head h reads key / value head h / (heads / kv_heads).
  * norm_mode: RMS norm of q and k before rotation — LP_QKNORM_NONE, LP_QKNORM_HEAD (over each head's dim, gains [dim] shared by the
@@ -730,7 +732,14 @@ typedef struct lp_window_attn_desc {
   int kv_shared;                            /* != 0: `cache` is another layer's, already written for this step's rows: lp_window_attn_prep
                                                prepares the queries only and qkv holds no keys or values */
   const float* q_temp;                      /* [heads] or NULL */
-  const float* dist_amp; const float* dist_rate;   /* [heads] each, or both NULL */
+  const float* dist_amp; const float* dist_rate;   /* [heads] each, or both NULL; dist_amp alone: the bias dist_amp[h] * (i - j) */
+  int v_is_k;                               /* != 0: the values are the cached keys: cache rows hold kv_heads * dim floats, vdim = dim, no v_off */
+  const float* gate; long long ldg;         /* [rows, heads * vdim] or NULL: out *= sigmoid(gate) (lp_window_attn, lp_window_attn_tiles) */
+  float out_scale;                          /* multiplies the output of the same two; 0 is taken as 1 */
+  float pos_temp_coef; int pos_temp_every;  /* every > 0: the query at position p is multiplied by 1 + coef ln(floor((p + 1) / every) + 1) */
+  const float* conv_w; int conv_taps;       /* one-token steps (each row the only one of its request): q and k (k_off = q_off + heads * dim)
+                                               first pass the causal convolution of lp_causal_conv_f32 without its input, */
+  const int* row_slot; float* conv_state; long long conv_stride;   /* w [taps][(heads + kv_heads) * dim], carried inputs in the row's slot */
 } lp_window_attn_desc;
 /* norm + rotation of the step's rows; keys and values go to the request's pages */
 int lp_window_attn_prep(const lp_window_attn_desc* desc, int R, const int* row_seq, const int* row_pos, void* stream);
@@ -792,6 +801,34 @@ size_t lp_mlstm_workspace_bytes(int rows, int heads, int vdim);
 int lp_mlstm(const lp_mlstm_desc* desc, int n_seqs, int R, const int* seq_row0, const int* seq_pos0, const int* seq_slot, void* workspace,
              size_t workspace_bytes, void* stream);
 
+/* Linear attention with a decay per key channel (csrc/lp_gla.cu).  Per head, from fp32 rows q, k [heads * dim], v [heads * vdim] (each
+ * with a row stride of its own): S_t = diag(a_t) S_(t-1) + k_t v_t^T, o_t = S_t^T (q_scale q_t) or, with bonus [heads * dim],
+ * o_t = (S_(t-1) + diag(bonus) k_t v_t^T)^T (q_scale q_t); out = o / rms(o) per head (eps) * out_gain[h * gain_stride + c] (NULL: none;
+ * gain_stride 0: one gain for all heads) * silu(gate) (NULL: none).  The decay a_t = exp(-exp(z)) or sigmoid(z)^decay_exp, z fp32
+ * [rows, ldz]; with z NULL it is made from z = w2 act(t) + z_bias, t fp32 [rows, rank], w2 bf16 [heads * dim, rank], act tanh when t_tanh
+ * (for one-token steps).  state fp32 [slots][heads][dim][vdim] (slot_stride elements per slot), carried between steps; a request at
+ * position 0 starts from zero without reading its slot.  Batch and chunk tables as for lp_retention_prefill; `longest`: the most rows
+ * one request brings (1: a one-token step, chunk tables unused). */
+enum lp_gla_decay { LP_GLA_DECAY_DOUBLE_EXP = 0, LP_GLA_DECAY_SIGMOID_POW = 1 };
+typedef struct lp_gla_desc {
+  const float* q; const float* k; const float* v; long long ldq, ldk, ldv;
+  int heads, dim, vdim; float q_scale;
+  int decay; float decay_exp;
+  const float* z; long long ldz;
+  const float* t; long long ldt; const void* w2; long long ldw2; int rank, t_tanh; const float* z_bias;
+  const float* bonus;
+  const float* out_gain; long long gain_stride; const float* gate; long long ldg; float eps;
+  float* state; long long slot_stride;
+  void* out; long long ldo; int out_fp32;
+} lp_gla_desc;
+size_t lp_gla_workspace_bytes(int n_chunks, int R, int longest, int heads, int dim, int vdim);
+int lp_gla(const lp_gla_desc* desc, int n_seqs, int n_chunks, int R, int longest, const int* seq_row0, const int* seq_pos0, const int* seq_slot,
+           const int* seq_chunk0, const int* chunk_seq, const int* chunk_row0, const int* chunk_len, void* workspace, size_t workspace_bytes,
+           void* stream);
+/* the operand of a low-rank product whose result must stay near fp32: out = act(t) (act_tanh: tanh) as fp32 [R, rank], or (split) as
+ * bf16 [R, 2 rank] = [hi | lo] with hi + lo ~ act(t), to be multiplied by a weight written twice side by side */
+int lp_lowrank_operand(const float* t, long long ldt, int R, int rank, int act_tanh, void* out, long long ldo, int split, void* stream);
+
 /* x[r, 2i] += sin(row_pos[r] * f_i), x[r, 2i + 1] += cos(...): absolute sinusoidal positions; freq fp32 [2][ceil(D / 2)] holds every
  * frequency as two floats, f_i = freq[0][i] + freq[1][i] (a float64 value split on the host) */
 int lp_add_positions_f32(float* x, long long ldx, int R, int D, const int* row_pos, const float* freq, void* stream);
@@ -803,12 +840,37 @@ int lp_token_shift_f32(const float* h, long long ldh, const float* mu, int R, in
                        const int* seq_row0, const int* seq_slot, float* state, long long slot_stride, void* out, long long ldo,
                        int out_fp32, void* stream);
 
-/* short causal convolution added to its input: out_t = h_t + sum_k w[k] * h_(t - taps + 1 + k) per channel, w fp32 [taps][D].  The taps - 1
+/* the token shift with n mixing vectors mu [n][D]: out[i][r] = h[r] + (h[r - 1] - h[r]) * mu[i], operand i starting i * mix_stride elements
+ * after out; rows and slot as for lp_token_shift_f32 */
+int lp_token_shift_mix_f32(const float* h, long long ldh, const float* mu, int n, int R, int D, const int* row_seq, const int* row_pos,
+                           const int* seq_row0, const int* seq_slot, float* state, long long slot_stride, void* out, long long ldo,
+                           long long mix_stride, int out_fp32, void* stream);
+
+/* out[r, s * D + c] = table[ids[r], c] * scale + pos_table[row_pos[r], c] for s < copies (pos_table bf16 [n_pos, ldp]; NULL: no positions) */
+int lp_embed_streams_f32(const int* ids, int R, const void* table, long long ldt, int vocab, float scale, const void* pos_table, long long ldp,
+                         int n_pos, const int* row_pos, float* out, long long ldo, int D, int copies, void* stream);
+/* Hyper-connections: a residual stream kept as n copies x_s (row m of x holds them side by side).  With y (NULL: nothing to close) every
+ * copy becomes x_t <- sum_s mix[s * n + t] x_s + out_w[t] y, all from the old ones; with gain (NULL: nothing to open) h receives the next
+ * operand, norm(u) = u / sqrt(mean(u^2) + eps) * gain of u = sum_s in_w[s] x_s over the new copies (in_w NULL: their plain sum).  With mu
+ * [n_mix][D] (one-token steps: row m is request m at row_pos[m], its slot row_slot[m]) h is n_mix operands, mix_stride elements apart, as
+ * lp_token_shift_mix_f32 makes them.  1 <= n <= lp_hyper_max_streams(). */
+typedef struct lp_hyper_desc {
+  float* x; long long ldx; int n, D;
+  const float* y; long long ldy; const float* mix; const float* out_w;
+  const float* in_w; const float* gain; float eps;
+  void* h; long long ldh; int h_fp32;
+  const float* mu; int n_mix; long long mix_stride;
+  const int* row_pos; const int* row_slot; float* state; long long slot_stride;
+} lp_hyper_desc;
+int lp_hyper_max_streams(void);
+int lp_hyper_f32(const lp_hyper_desc* desc, int M, void* stream);
+
+/* short causal convolution: out_t = (add_input: h_t +) sum_k w[k] * h_(t - taps + 1 + k) per channel, w fp32 [taps][D].  The taps - 1
  * inputs before a request's first row of the step are the request's slot of `state` (taps - 1 rows of D, oldest first; zeros before
  * position 0), which afterwards holds the request's last taps - 1 inputs.  The chunk tables are those of lp_retention_prefill, longest_chunk
  * the most rows one of them has.  1 <= taps <= lp_causal_conv_max_taps() (with one tap there is no state).  Not in place. */
 int lp_causal_conv_max_taps(void);
-int lp_causal_conv_f32(const float* h, long long ldh, const float* w, int taps, int D, int n_chunks, const int* chunk_seq,
+int lp_causal_conv_f32(const float* h, long long ldh, const float* w, int taps, int add_input, int D, int n_chunks, const int* chunk_seq,
                        const int* chunk_row0, const int* chunk_len, int longest_chunk, const int* row_pos, const int* seq_row0,
                        const int* seq_slot, float* state, long long slot_stride, void* out, long long ldo, int out_fp32, void* stream);
 /* the norm after the residual sum, in place: x <- z / sqrt(mean(z^2) + eps) * gain[c] with z = alpha x + y.  `out` (NULL: none) receives
@@ -828,6 +890,11 @@ int lp_moe_route(const void* h, long long ldh, int h_fp32, int T, int D, const v
  * weights = softmax over the chosen logits only */
 int lp_moe_route_softmax(const void* h, long long ldh, int h_fp32, int T, int D, const void* w_router, long long ldw, int E,
                          const float* logit_bias, int top, int* idx_out, float* w_out, void* stream);
+/* softmax scores over groups of experts: s = softmax(W_router h), a group's score is its largest s, only the keep_groups best of n_groups
+ * equal groups of neighbours stay eligible, the `top` largest eligible s are chosen (ties to the lower index), weights = the chosen s /
+ * (their sum + 1e-20) * w_scale */
+int lp_moe_route_group_softmax(const void* h, long long ldh, int h_fp32, int T, int D, const void* w_router, long long ldw, int E, int n_groups,
+                               int keep_groups, int top, float w_scale, int* idx_out, float* w_out, void* stream);
 /* the plain sigmoid router: scores = sigmoid(W_router h), the `top` largest are chosen (ties to the lower index), weights = the chosen
  * scores as they are */
 int lp_moe_route_sigmoid(const void* h, long long ldh, int h_fp32, int T, int D, const void* w_router, long long ldw, int E, int top,

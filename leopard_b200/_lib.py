@@ -79,10 +79,12 @@ _P = C.POINTER
 
 EPI_NONE, EPI_XIELU, EPI_SILU_GATE, EPI_RELU2, EPI_CLAMP_GLU, EPI_GELU_GATE = 0, 1, 2, 3, 4, 5
 GATED_EPIS = (EPI_SILU_GATE, EPI_CLAMP_GLU, EPI_GELU_GATE)      # W = [gate rows; up rows], half as many output columns
+GLA_DECAY_DOUBLE_EXP, GLA_DECAY_SIGMOID_POW = 0, 1
 RET_FINISH_GATED_NORM, RET_FINISH_RAW = 0, 1
 QKNORM_NONE, QKNORM_HEAD, QKNORM_FULL = 0, 1, 2
 ROT_HALF, ROT_INTERLEAVED = 0, 1
 RETENTION_CHUNK = 32
+LINEAR_ROWS_MAX, LINEAR_ROWS_COLS = 8, 8      # lp_linear: up to this many rows stream the weights, a CTA to so many columns
 
 
 class LinearDesc(C.Structure):
@@ -90,7 +92,7 @@ class LinearDesc(C.Structure):
     _fields_ = [("A", _vp), ("lda", _ll), ("a_batch", _ll), ("a_fp32", _i), ("W", _vp), ("ldw", _ll), ("w_batch", _ll), ("C", _vp),
                 ("ldc", _ll), ("c_batch", _ll), ("c_fp32", _i), ("M", _i), ("N", _i), ("K", _i), ("batch", _i), ("epi", _i),
                 ("epi_a", _f), ("epi_b", _f), ("c_accum", _i), ("c_scale", _f), ("bias", _vp), ("row_scale", _vp), ("gate", _vp), ("ldg", _ll),
-                ("gate_batch", _ll)]
+                ("gate_batch", _ll), ("seg_cols", _i), ("n_segs", _i), ("a_seg", _ll)]
 
 
 class WindowAttnDesc(C.Structure):
@@ -101,7 +103,9 @@ class WindowAttnDesc(C.Structure):
                 ("page_size", _i), ("page_table", _vp), ("max_pages", _i), ("pooled", _vp), ("pooled_table", _vp),
                 ("max_pooled_pages", _i), ("pool", _i), ("window", _i), ("keep_first", _i), ("scale", _f), ("softcap", _f), ("sink", _i),
                 ("q_bias", _vp), ("k_bias", _vp), ("v_bias", _vp), ("v_norm", _i), ("talk", _vp), ("g_off", _i), ("chunk", _i), ("kv_shared", _i),
-                ("q_temp", _vp), ("dist_amp", _vp), ("dist_rate", _vp)]
+                ("q_temp", _vp), ("dist_amp", _vp), ("dist_rate", _vp), ("v_is_k", _i), ("gate", _vp), ("ldg", _ll), ("out_scale", _f),
+                ("pos_temp_coef", _f), ("pos_temp_every", _i), ("conv_w", _vp), ("conv_taps", _i), ("row_slot", _vp), ("conv_state", _vp),
+                ("conv_stride", _ll)]
 
 
 class MinGRUDesc(C.Structure):
@@ -131,6 +135,21 @@ class MLSTMDesc(C.Structure):
     _fields_ = [("proj", _vp), ("ld", _ll), ("q_off", _i), ("k_off", _i), ("v_off", _i), ("g_off", _i), ("i_off", _i), ("f_off", _i),
                 ("heads", _i), ("dim", _i), ("vdim", _i), ("i_bias", _vp), ("f_bias", _vp), ("gate_cap", _f), ("q_scale", _f),
                 ("eps", _f), ("out_gain", _vp), ("state", _vp), ("slot_stride", _ll), ("out", _vp), ("ldo", _ll), ("out_fp32", _i)]
+
+
+class GlaDesc(C.Structure):
+    """lp_gla_desc (include/leopard_b200.h)."""
+    _fields_ = [("q", _vp), ("k", _vp), ("v", _vp), ("ldq", _ll), ("ldk", _ll), ("ldv", _ll), ("heads", _i), ("dim", _i), ("vdim", _i),
+                ("q_scale", _f), ("decay", _i), ("decay_exp", _f), ("z", _vp), ("ldz", _ll), ("t", _vp), ("ldt", _ll), ("w2", _vp),
+                ("ldw2", _ll), ("rank", _i), ("t_tanh", _i), ("z_bias", _vp), ("bonus", _vp), ("out_gain", _vp), ("gain_stride", _ll),
+                ("gate", _vp), ("ldg", _ll), ("eps", _f), ("state", _vp), ("slot_stride", _ll), ("out", _vp), ("ldo", _ll), ("out_fp32", _i)]
+
+
+class HyperDesc(C.Structure):
+    """lp_hyper_desc (include/leopard_b200.h)."""
+    _fields_ = [("x", _vp), ("ldx", _ll), ("n", _i), ("D", _i), ("y", _vp), ("ldy", _ll), ("mix", _vp), ("out_w", _vp), ("in_w", _vp),
+                ("gain", _vp), ("eps", _f), ("h", _vp), ("ldh", _ll), ("h_fp32", _i), ("mu", _vp), ("n_mix", _i), ("mix_stride", _ll),
+                ("row_pos", _vp), ("row_slot", _vp), ("state", _vp), ("slot_stride", _ll)]
 
 
 # name -> (restype, argtypes); must list EVERY symbol include/leopard_b200.h declares (tests/test_abi.py checks)
@@ -236,7 +255,15 @@ _SIGS = {
     "lp_add_row_f32": (_i, [_vp, _ll, _vp, _i, _i, _vp]),
     "lp_token_shift_f32": (_i, [_vp, _ll, _vp, _i, _i, _vp, _vp, _vp, _vp, _vp, _ll, _vp, _ll, _i, _vp]),
     "lp_causal_conv_max_taps": (_i, []),
-    "lp_causal_conv_f32": (_i, [_vp, _ll, _vp, _i, _i, _i, _vp, _vp, _vp, _i, _vp, _vp, _vp, _vp, _ll, _vp, _ll, _i, _vp]),
+    "lp_gla_workspace_bytes": (_sz, [_i, _i, _i, _i, _i, _i]),
+    "lp_gla": (_i, [C.POINTER(GlaDesc), _i, _i, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _sz, _vp]),
+    "lp_lowrank_operand": (_i, [_vp, _ll, _i, _i, _i, _vp, _ll, _i, _vp]),
+    "lp_token_shift_mix_f32": (_i, [_vp, _ll, _vp, _i, _i, _i, _vp, _vp, _vp, _vp, _vp, _ll, _vp, _ll, _ll, _i, _vp]),
+    "lp_embed_streams_f32": (_i, [_vp, _i, _vp, _ll, _i, _f, _vp, _ll, _i, _vp, _vp, _ll, _i, _i, _vp]),
+    "lp_hyper_max_streams": (_i, []),
+    "lp_hyper_f32": (_i, [C.POINTER(HyperDesc), _i, _vp]),
+    "lp_moe_route_group_softmax": (_i, [_vp, _ll, _i, _i, _i, _vp, _ll, _i, _i, _i, _i, _f, _vp, _vp, _vp]),
+    "lp_causal_conv_f32": (_i, [_vp, _ll, _vp, _i, _i, _i, _i, _vp, _vp, _vp, _i, _vp, _vp, _vp, _vp, _ll, _vp, _ll, _i, _vp]),
     "lp_post_norm_f32": (_i, [_vp, _ll, _vp, _ll, _f, _i, _i, _vp, _f, _vp, _ll, _i, _vp, _i, _vp, _vp, _vp, _ll, _vp]),
     "lp_moe_route_softmax": (_i, [_vp, _ll, _i, _i, _i, _vp, _ll, _i, _vp, _i, _vp, _vp, _vp]),
     "lp_mingru_workspace_bytes": (_sz, [_i, _i]),
@@ -298,7 +325,7 @@ def lib():
     return _lib
 
 
-# ---- the 32-bit residual-stream entry points (csrc/lp_linear.cu, lp_stream32.cu, lp_seqmix.cu, lp_winattn.cu, lp_mingru.cu, lp_mlstm.cu, lp_moe.cu) -----------------------------------
+# ---- the 32-bit residual-stream entry points (csrc/lp_linear.cu, lp_stream32.cu, lp_seqmix.cu, lp_winattn.cu, lp_mingru.cu, lp_mlstm.cu, lp_gla.cu, lp_moe.cu) -----------------------------------
 # They need none of the tcgen05 translation units, so a model that uses only them can run from a library of its own that compiles in
 # seconds (build.build_native("stream32")); the full library contains the same symbols and is preferred when it is already built.
 STREAM32_LIB_PATH = PKG / "lib" / "libleopard_stream32.so"
@@ -310,7 +337,9 @@ STREAM32_SYMBOLS = ("lp_last_error", "lp_abi_version", "lp_launch_count", "lp_li
                     "lp_mingru_prefill", "lp_mingru_decode", "lp_window_attn_talk", "lp_window_attn_talk_tiles", "lp_mlstm_workspace_bytes", "lp_mlstm",
                     "lp_add_positions_f32", "lp_add_row_f32", "lp_token_shift_f32", "lp_moe_route_softmax", "lp_glu_scaled_f32", "lp_dyt_f32",
                     "lp_rmsnorm_gated_f32", "lp_gated_axpy_f32", "lp_depth_average_f32", "lp_moe_route_sigmoid", "lp_moe_sorted_weights",
-                    "lp_causal_conv_max_taps", "lp_causal_conv_f32", "lp_post_norm_f32", "lp_latent_attend_tiles")
+                    "lp_causal_conv_max_taps", "lp_causal_conv_f32", "lp_post_norm_f32", "lp_latent_attend_tiles", "lp_gla_workspace_bytes", "lp_gla",
+                    "lp_lowrank_operand", "lp_token_shift_mix_f32", "lp_embed_streams_f32", "lp_hyper_max_streams", "lp_hyper_f32",
+                    "lp_moe_route_group_softmax")
 STREAM32_OPTIONAL = ("lp_gemm_bf16",)      # present in the native libraries, absent from the CPU-emulated build
 _stream32 = None
 

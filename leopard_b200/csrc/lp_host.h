@@ -30,6 +30,25 @@ const char* get_error();
 
 int sm_count();
 
+#ifdef __CUDACC__
+// two fp32 multiply-adds (products) in one instruction
+__device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
+  float2 d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;"
+      : "=l"(reinterpret_cast<unsigned long long&>(d))
+      : "l"(reinterpret_cast<const unsigned long long&>(a)), "l"(reinterpret_cast<const unsigned long long&>(b)),
+        "l"(reinterpret_cast<const unsigned long long&>(c)));
+  return d;
+}
+__device__ __forceinline__ float2 mul2(float2 a, float2 b) {
+  float2 d;
+  asm("mul.rn.f32x2 %0, %1, %2;"
+      : "=l"(reinterpret_cast<unsigned long long&>(d))
+      : "l"(reinterpret_cast<const unsigned long long&>(a)), "l"(reinterpret_cast<const unsigned long long&>(b)));
+  return d;
+}
+#endif
+
 // prefill kernels are launched with the programmatic-dependent-launch attribute when this is on (lp_set_prefill_pdl):
 // every such kernel calls griddepcontrol.wait before its first dependent global access
 bool prefill_pdl();

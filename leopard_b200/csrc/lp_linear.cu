@@ -8,7 +8,8 @@
 //                      that multiplies its first products) and take a bias per weight row.  With c_accum the result is scaled
 //                      and ADDED to C (the residual update of a pre-norm layer); with `gate` it is first multiplied by
 //                      sigmoid(gate[m, n]) (a gated residual branch closes in the store of its last product).
-//                      `batch` independent problems with element strides (per-head products of latent attention).
+//                      seg_cols: groups of output columns that read operands of their own (a mixer whose projections see different
+//                      mixes of the stream) in one launch.  `batch` independent problems with element strides (per-head products of latent attention).
 //                      Two kernels: a 64 x 64 x 16 shared-memory tile kernel (prefill), and a weight-streaming kernel with one warp
 //                      per output column for M <= 8 rows (decode: every weight byte is read once, 16-byte loads).
 //   lp_linear_grouped  the same tile kernel over row tiles that each belong to one group (expert): tile t multiplies rows
@@ -39,8 +40,16 @@ struct LinArgs {
   int a_div;
   const float* bias;      // [N] added to the accumulators before the epilogue, or NULL
   const float* row_scale; // [rows of C] multiplies the accumulators before the bias, or NULL
+  int seg_cols, n_segs; long long a_seg;   // seg_cols > 0: output columns [i seg_cols, (i + 1) seg_cols) read A + i a_seg (the last of n_segs: all that follow)
   const float* gate; long long ldg, gate_batch;   // [rows of C, N'] pre-activations: the result is multiplied by sigmoid(gate), or NULL
 };
+
+// elements between A and the operand of the columns from n on
+__device__ __forceinline__ long long lin_seg(const LinArgs& a, int n) {
+  if (a.seg_cols <= 0) return 0;
+  const int i = n / a.seg_cols;
+  return (long long)(i < a.n_segs ? i : a.n_segs - 1) * a.a_seg;
+}
 
 __device__ __forceinline__ float lin_load(const float* p) { return *p; }
 __device__ __forceinline__ float lin_load(const bf16* p) { return __bfloat162float(*p); }
@@ -100,7 +109,7 @@ __global__ void __launch_bounds__(LIN_THREADS) linear_tile_kernel(LinArgs a) {
     if (group < 0) return;
   }
   const int n_out = GATED ? a.N / 2 : a.N;
-  const AT* A = reinterpret_cast<const AT*>(a.A) + (long long)z_id * a.a_batch;
+  const AT* A = reinterpret_cast<const AT*>(a.A) + (long long)z_id * a.a_batch + lin_seg(a, tile_n * LIN_BN);
   const bf16* W = a.W + (long long)(z_id + group) * a.w_batch;   // grouped launches have one batch: z_id = 0
   CT* C = reinterpret_cast<CT*>(a.C) + (long long)z_id * a.c_batch;
   const int m0 = tile_m * LIN_BM, n0 = tile_n * LIN_BN;
@@ -186,7 +195,8 @@ __global__ void __launch_bounds__(ROWS_WARPS * 32) linear_rows_kernel(LinArgs a)
   const bool active = n < n_out;
   const bool pairs = a.z_group != nullptr;
   const int M = pairs ? 1 : a.M;
-  const AT* A = reinterpret_cast<const AT*>(a.A) + (pairs ? (long long)(z / a.a_div) * a.lda : (long long)z * a.a_batch);
+  const AT* A = reinterpret_cast<const AT*>(a.A) + (pairs ? (long long)(z / a.a_div) * a.lda : (long long)z * a.a_batch) +
+                lin_seg(a, blockIdx.x * ROWS_WARPS);
   const bf16* W = a.W + (long long)(pairs ? a.z_group[z] : z) * a.w_batch;
   CT* C = reinterpret_cast<CT*>(a.C) + (pairs ? (long long)z * a.ldc : (long long)z * a.c_batch);
   const bf16* w1 = W + (long long)(active ? n : 0) * a.ldw;
@@ -323,7 +333,12 @@ extern "C" int lp_linear(const lp_linear_desc* d, void* stream_) {
   a.epi = d->epi; a.e0 = d->epi_a; a.e1 = d->epi_b; a.c_accum = d->c_accum; a.c_scale = d->c_scale;
   a.a_rows = nullptr; a.tile_group = nullptr; a.z_group = nullptr; a.a_div = 1;
   a.bias = d->bias; a.row_scale = d->row_scale; a.gate = d->gate; a.ldg = d->ldg; a.gate_batch = d->gate_batch;
+  a.seg_cols = d->seg_cols; a.n_segs = d->n_segs; a.a_seg = d->a_seg;
   LP_REQUIRE(d->batch == 1 || (d->bias == nullptr && d->row_scale == nullptr), "lp_linear: bias and row scale are for one problem");
+  // a CTA's columns read one operand: 8 columns for few rows, a tile otherwise
+  LP_REQUIRE(d->seg_cols == 0 || (d->seg_cols > 0 && d->n_segs >= 1 && d->seg_cols % (d->M <= ROWS_MAX ? ROWS_WARPS : LIN_BN) == 0),
+             "lp_linear: column segments of %d do not fit the CTAs of a product of %d rows", d->seg_cols, d->M);
+  LP_REQUIRE(d->seg_cols == 0 || !gated_epi(d->epi), "lp_linear: a gated unit has one operand");
   return dispatch_linear(a, d->a_fp32, d->c_fp32, d->batch, (d->M + LIN_BM - 1) / LIN_BM, true, stream);
 }
 
@@ -345,6 +360,7 @@ extern "C" int lp_linear_pairs(const lp_linear_desc* d, const int* pair_group, i
   a.epi = d->epi; a.e0 = d->epi_a; a.e1 = d->epi_b; a.c_accum = d->c_accum; a.c_scale = d->c_scale;
   a.a_rows = nullptr; a.tile_group = nullptr; a.z_group = pair_group; a.a_div = a_div;
   a.bias = d->bias; a.row_scale = d->row_scale; a.gate = d->gate; a.ldg = d->ldg; a.gate_batch = d->gate_batch;
+  a.seg_cols = 0; a.n_segs = 0; a.a_seg = 0;
   return dispatch_linear(a, d->a_fp32, d->c_fp32, n_pairs, 1, true, stream);
 }
 
@@ -364,6 +380,7 @@ extern "C" int lp_linear_grouped(const lp_linear_desc* d, const int* tile_group,
   a.epi = d->epi; a.e0 = d->epi_a; a.e1 = d->epi_b; a.c_accum = d->c_accum; a.c_scale = d->c_scale;
   a.a_rows = a_rows; a.tile_group = tile_group; a.z_group = nullptr; a.a_div = 1;
   a.bias = d->bias; a.row_scale = d->row_scale; a.gate = d->gate; a.ldg = d->ldg; a.gate_batch = d->gate_batch;
+  a.seg_cols = 0; a.n_segs = 0; a.a_seg = 0;
   return dispatch_linear(a, d->a_fp32, d->c_fp32, 1, n_tiles, false, stream);
 }
 

@@ -8,6 +8,8 @@
 //                    Optionally one more row of weights gives a per-token sigmoid gate (for a shared expert).
 //   lp_moe_route_softmax  the plain token-choice router on the same kernel: logits z = W_router h + bias, the `top` largest logits are
 //                    chosen (ties to the lower index), weights = softmax over the chosen logits only.
+//   lp_moe_route_group_softmax  softmax scores over all experts, a group counts by its largest score, weights = chosen scores over their sum
+//                    times a constant.
 //   lp_moe_route_sigmoid  the plain sigmoid router on the same kernel: the `top` largest scores sigmoid(z) are chosen and are the
 //                    weights as they are (for designs that multiply an expert's INPUT by its score: lp_moe_sorted_weights puts the
 //                    weights into the row space of lp_moe_align, the grouped products take them as row scales).
@@ -22,7 +24,7 @@ namespace lp {
 
 typedef __nv_bfloat16 bf16;
 
-constexpr int MOE_MAX_EXPERTS = 512;
+constexpr int MOE_MAX_EXPERTS = 512, MOE_MAX_GROUPS = 64;
 constexpr int ROUTE_WARPS = 8;
 
 // eight bf16 values of a 16-byte load -> fp32 (a bf16 is the upper half of an fp32)
@@ -37,16 +39,31 @@ template <typename HT> __device__ __forceinline__ float moe_ld(const HT* p);
 template <> __device__ __forceinline__ float moe_ld<float>(const float* p) { return *p; }
 template <> __device__ __forceinline__ float moe_ld<bf16>(const bf16* p) { return __bfloat162float(*p); }
 
+// the largest value of the warp's candidates, the lower index among equals; a lane without a candidate brings index `none`
+__device__ __forceinline__ void warp_best(float& v, int& i, int none) {
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    const float ov = __shfl_xor_sync(0xffffffffu, v, o);
+    const int oi = __shfl_xor_sync(0xffffffffu, i, o);
+    if (oi != none && (i == none || ov > v || (ov == v && oi < i))) {
+      v = ov;
+      i = oi;
+    }
+  }
+}
+
 // One CTA per token: the warps share out the router rows (and the gate row), 16-byte loads of the bf16 weights when the width
-// allows; then one thread makes the choice among the E scores.
+// allows; then one warp makes the choice among the E scores.
 template <typename HT>
 __global__ void __launch_bounds__(ROUTE_WARPS * 32)
 moe_route_kernel(const HT* __restrict__ h, long long ldh, int T, int D, const bf16* __restrict__ w_router, long long ldw, int E,
                  const float* __restrict__ correction, int n_groups, int keep_groups, int top, const bf16* __restrict__ w_gate,
                  int* __restrict__ idx_out, float* __restrict__ w_out, float* __restrict__ gate_out, int softmax_mode,
-                 const float* __restrict__ logit_bias) {
+                 const float* __restrict__ logit_bias, float w_scale) {
   __shared__ float sc[MOE_MAX_EXPERTS];   // sigmoid scores
   __shared__ float ch[MOE_MAX_EXPERTS];   // choice scores (minus infinity once taken or not eligible)
+  __shared__ float gsc[MOE_MAX_GROUPS];   // group scores
+  __shared__ int kept[MOE_MAX_GROUPS];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x;
   if (t >= T) return;
@@ -71,7 +88,7 @@ moe_route_kernel(const HT* __restrict__ h, long long ldh, int T, int D, const bf
     for (int o = 16; o > 0; o >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
     const float s = 1.0f / (1.0f + expf(-acc));
     if (lane == 0) {
-      if (softmax_mode == 1) {      // the logit itself is score and choice
+      if (softmax_mode == 1 || softmax_mode == 3) {      // the logit itself is score and choice
         sc[e] = ch[e] = acc + (logit_bias != nullptr ? logit_bias[e] : 0.f);
       } else if (e < E) {
         sc[e] = s;
@@ -82,60 +99,67 @@ moe_route_kernel(const HT* __restrict__ h, long long ldh, int T, int D, const bf
     }
   }
   __syncthreads();
-  if (threadIdx.x != 0) return;
+  if (warp != 0) return;
+  // the choice is the first warp's: every lane looks after the experts (and groups) lane, lane + 32, ...
+  if (softmax_mode == 3) {      // scores: softmax over all experts
+    float mx = -INFINITY, sum = 0.f;
+    for (int e = lane; e < E; e += 32) mx = fmaxf(mx, sc[e]);
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+    for (int e = lane; e < E; e += 32) sum += expf(sc[e] - mx);
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+    for (int e = lane; e < E; e += 32) sc[e] = ch[e] = expf(sc[e] - mx) / sum;
+    __syncwarp();
+  }
   if (n_groups > 1 && keep_groups < n_groups) {
     const int gs = E / n_groups;
-    // group score: the sum of the two largest choice scores (of the only one when groups hold a single expert)
-    float gscore[64];
-    for (int g = 0; g < n_groups; ++g) {
+    // group score: the largest choice score (mode 3), or the sum of the two largest (of the only one when groups hold a single expert)
+    for (int g = lane; g < n_groups; g += 32) {
       float a = -INFINITY, b = -INFINITY;
       for (int i = 0; i < gs; ++i) {
         const float v = ch[g * gs + i];
         if (v > a) { b = a; a = v; } else if (v > b) { b = v; }
       }
-      gscore[g] = gs >= 2 ? a + b : a;
+      gsc[g] = gs >= 2 && softmax_mode != 3 ? a + b : a;
+      kept[g] = 0;
     }
-    // keep the best groups: mark the others
-    bool kept[64];
-    for (int g = 0; g < n_groups; ++g) kept[g] = false;
-    for (int k = 0; k < keep_groups; ++k) {
-      int best = -1;
-      for (int g = 0; g < n_groups; ++g)
-        if (!kept[g] && (best < 0 || gscore[g] > gscore[best])) best = g;
-      kept[best] = true;
+    __syncwarp();
+    for (int k = 0; k < keep_groups; ++k) {      // keep the best groups, the others lose their experts
+      float v = -INFINITY;
+      int best = n_groups;
+      for (int g = lane; g < n_groups; g += 32)
+        if (!kept[g] && (best == n_groups || gsc[g] > v)) { v = gsc[g]; best = g; }
+      warp_best(v, best, n_groups);
+      if (lane == 0) kept[best] = 1;
+      __syncwarp();
     }
-    for (int g = 0; g < n_groups; ++g)
-      if (!kept[g])
-        for (int i = 0; i < gs; ++i) ch[g * gs + i] = -INFINITY;
+    for (int e = lane; e < E; e += 32)
+      if (!kept[e / gs]) ch[e] = -INFINITY;
+    __syncwarp();
   }
-  if (softmax_mode == 1) {
-    float mx = -INFINITY, sum = 0.f;
-    for (int k = 0; k < top; ++k) {
-      int best = 0;
-      for (int e = 1; e < E; ++e)
-        if (ch[e] > ch[best]) best = e;
-      idx_out[(long long)t * top + k] = best;
-      if (k == 0) mx = sc[best];      // the first choice is the largest logit
-      const float p = expf(sc[best] - mx);
-      w_out[(long long)t * top + k] = p;
-      sum += p;
-      ch[best] = -INFINITY;
-    }
-    for (int k = 0; k < top; ++k) w_out[(long long)t * top + k] /= sum;
-    return;
-  }
-  float sum = 0.f;
+  float sum = 0.f, first = 0.f;
   for (int k = 0; k < top; ++k) {
-    int best = 0;
-    for (int e = 1; e < E; ++e)
-      if (ch[e] > ch[best]) best = e;
-    idx_out[(long long)t * top + k] = best;
-    sum += sc[best];
-    ch[best] = -INFINITY;   // taken; the host guarantees that the eligible experts outnumber `top`
+    float v = -INFINITY;
+    int best = E;
+    for (int e = lane; e < E; e += 32)
+      if (ch[e] > v) { v = ch[e]; best = e; }
+    warp_best(v, best, E);
+    if (best >= E) best = 0;      // nothing finite is left (not a number in the logits); the host guarantees enough eligible experts
+    const float s = sc[best];
+    if (k == 0) first = s;        // mode 1: the first choice is the largest logit
+    const float p = softmax_mode == 1 ? expf(s - first) : s;
+    sum += p;
+    if (lane == 0) {
+      idx_out[(long long)t * top + k] = best;
+      w_out[(long long)t * top + k] = p;
+      ch[best] = -INFINITY;       // taken
+    }
+    __syncwarp();
   }
-  // softmax_mode 2: the chosen scores as they are
-  for (int k = 0; k < top; ++k)
-    w_out[(long long)t * top + k] = sc[idx_out[(long long)t * top + k]] / (softmax_mode == 2 ? 1.0f : sum + 1e-20f);
+  // modes: 0, 3 scores over their sum; 1 softmax over the chosen logits; 2 the chosen scores as they are
+  const float scale = softmax_mode == 2 ? 1.0f : softmax_mode == 1 ? 1.0f / sum : w_scale / (sum + 1e-20f);
+  for (int k = lane; k < top; k += 32) w_out[(long long)t * top + k] *= scale;
 }
 
 __global__ void moe_sorted_weights_kernel(const int* __restrict__ pair_row, const float* __restrict__ w, int n_pairs, float* __restrict__ sorted) {
@@ -210,11 +234,11 @@ extern "C" int lp_moe_route(const void* h, long long ldh, int h_fp32, int T, int
   if (h_fp32)
     moe_route_kernel<float><<<grid, ROUTE_WARPS * 32, 0, stream>>>(reinterpret_cast<const float*>(h), ldh, T, D,
         reinterpret_cast<const bf16*>(w_router), ldw, E, correction, n_groups, keep_groups, top, reinterpret_cast<const bf16*>(w_gate),
-        idx_out, w_out, gate_out, 0, nullptr);
+        idx_out, w_out, gate_out, 0, nullptr, 1.0f);
   else
     moe_route_kernel<bf16><<<grid, ROUTE_WARPS * 32, 0, stream>>>(reinterpret_cast<const bf16*>(h), ldh, T, D,
         reinterpret_cast<const bf16*>(w_router), ldw, E, correction, n_groups, keep_groups, top, reinterpret_cast<const bf16*>(w_gate),
-        idx_out, w_out, gate_out, 0, nullptr);
+        idx_out, w_out, gate_out, 0, nullptr, 1.0f);
   note_launch();
   LP_CHECK_CUDA(cudaGetLastError());
   return 0;
@@ -230,10 +254,10 @@ extern "C" int lp_moe_route_softmax(const void* h, long long ldh, int h_fp32, in
   const unsigned grid = (unsigned)T;
   if (h_fp32)
     moe_route_kernel<float><<<grid, ROUTE_WARPS * 32, 0, stream>>>(reinterpret_cast<const float*>(h), ldh, T, D,
-        reinterpret_cast<const bf16*>(w_router), ldw, E, nullptr, 1, 1, top, nullptr, idx_out, w_out, nullptr, 1, logit_bias);
+        reinterpret_cast<const bf16*>(w_router), ldw, E, nullptr, 1, 1, top, nullptr, idx_out, w_out, nullptr, 1, logit_bias, 1.0f);
   else
     moe_route_kernel<bf16><<<grid, ROUTE_WARPS * 32, 0, stream>>>(reinterpret_cast<const bf16*>(h), ldh, T, D,
-        reinterpret_cast<const bf16*>(w_router), ldw, E, nullptr, 1, 1, top, nullptr, idx_out, w_out, nullptr, 1, logit_bias);
+        reinterpret_cast<const bf16*>(w_router), ldw, E, nullptr, 1, 1, top, nullptr, idx_out, w_out, nullptr, 1, logit_bias, 1.0f);
   note_launch();
   LP_CHECK_CUDA(cudaGetLastError());
   return 0;
@@ -249,10 +273,34 @@ extern "C" int lp_moe_route_sigmoid(const void* h, long long ldh, int h_fp32, in
   const unsigned grid = (unsigned)T;
   if (h_fp32)
     moe_route_kernel<float><<<grid, ROUTE_WARPS * 32, 0, stream>>>(reinterpret_cast<const float*>(h), ldh, T, D,
-        reinterpret_cast<const bf16*>(w_router), ldw, E, nullptr, 1, 1, top, nullptr, idx_out, w_out, nullptr, 2, nullptr);
+        reinterpret_cast<const bf16*>(w_router), ldw, E, nullptr, 1, 1, top, nullptr, idx_out, w_out, nullptr, 2, nullptr, 1.0f);
   else
     moe_route_kernel<bf16><<<grid, ROUTE_WARPS * 32, 0, stream>>>(reinterpret_cast<const bf16*>(h), ldh, T, D,
-        reinterpret_cast<const bf16*>(w_router), ldw, E, nullptr, 1, 1, top, nullptr, idx_out, w_out, nullptr, 2, nullptr);
+        reinterpret_cast<const bf16*>(w_router), ldw, E, nullptr, 1, 1, top, nullptr, idx_out, w_out, nullptr, 2, nullptr, 1.0f);
+  note_launch();
+  LP_CHECK_CUDA(cudaGetLastError());
+  return 0;
+}
+
+extern "C" int lp_moe_route_group_softmax(const void* h, long long ldh, int h_fp32, int T, int D, const void* w_router, long long ldw, int E,
+                                          int n_groups, int keep_groups, int top, float w_scale, int* idx_out, float* w_out, void* stream_) {
+  cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
+  LP_REQUIRE(h != nullptr && w_router != nullptr && idx_out != nullptr && w_out != nullptr, "lp_moe_route_group_softmax: null operand");
+  LP_REQUIRE(E > 0 && E <= MOE_MAX_EXPERTS && top > 0 && top <= E, "lp_moe_route_group_softmax: experts=%d top=%d (at most %d experts)", E, top,
+             MOE_MAX_EXPERTS);
+  LP_REQUIRE(n_groups >= 1 && n_groups <= E && E % n_groups == 0 && keep_groups >= 1 && keep_groups <= n_groups &&
+                 (n_groups <= MOE_MAX_GROUPS || keep_groups == n_groups),
+             "lp_moe_route_group_softmax: groups=%d keep=%d must divide experts=%d (at most %d groups)", n_groups, keep_groups, E, MOE_MAX_GROUPS);
+  LP_REQUIRE(keep_groups * (E / n_groups) >= top, "lp_moe_route_group_softmax: %d kept groups of %d experts cannot supply top=%d", keep_groups,
+             E / n_groups, top);
+  if (T <= 0) return 0;
+  const unsigned grid = (unsigned)T;
+  if (h_fp32)
+    moe_route_kernel<float><<<grid, ROUTE_WARPS * 32, 0, stream>>>(reinterpret_cast<const float*>(h), ldh, T, D,
+        reinterpret_cast<const bf16*>(w_router), ldw, E, nullptr, n_groups, keep_groups, top, nullptr, idx_out, w_out, nullptr, 3, nullptr, w_scale);
+  else
+    moe_route_kernel<bf16><<<grid, ROUTE_WARPS * 32, 0, stream>>>(reinterpret_cast<const bf16*>(h), ldh, T, D,
+        reinterpret_cast<const bf16*>(w_router), ldw, E, nullptr, n_groups, keep_groups, top, nullptr, idx_out, w_out, nullptr, 3, nullptr, w_scale);
   note_launch();
   LP_CHECK_CUDA(cudaGetLastError());
   return 0;

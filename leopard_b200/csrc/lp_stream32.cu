@@ -8,11 +8,16 @@
 //   lp_axpy_f32         y <- y + alpha x, the residual update after such a product.
 //   lp_add_positions_f32  x[r, 2i] += sin(p f_i), x[r, 2i + 1] += cos(p f_i) with p the row's position: absolute sinusoidal positions
 //                       added to the stream (fp32 angles with the product's rounding error carried along, accurate sincosf).
+//   lp_embed_streams_f32  x[r, s, :] = table[ids[r], :] * scale + pos[p, :]: the embedding with learned positions, written as every copy of a
+//                       stream that is kept several times (hyper-connections).
+//   lp_hyper_f32        closes one sublayer of a hyper-connected layer, x_t <- sum_s mix[s, t] x_s + out[t] y, and opens the next one, h =
+//                       norm(sum_s in[s] x_s), in one pass over the copies; in one-token steps also the token-shifted mixes of h.
+//   lp_token_shift_mix_f32  the token shift with several mixing vectors at once: one operand per vector from one read of the rows.
 //   lp_add_row_f32      x[r, :] += v for every row (a learned vector that marks a pass of a looped stack).
 //   lp_token_shift_f32  y_t = h_t + (h_(t-1) - h_t) * mu per channel, with h the rows as they came in; the row before a request's
 //                       first row of this step comes from the request's slot (zeros at position 0), and the slot then takes the
 //                       request's last row.
-//   lp_causal_conv_f32  out_t = h_t + sum_j w_j h_(t - K + 1 + j) per channel: a short causal convolution added to its input; the K - 1
+//   lp_causal_conv_f32  out_t = (h_t +) sum_j w_j h_(t - K + 1 + j) per channel: a short causal convolution, added to its input when asked; the K - 1
 //                       inputs before a request's first row of this step come from the request's slot (zeros before position 0), and
 //                       the slot then takes the request's last K - 1 inputs.
 //   lp_post_norm_f32    x <- norm(alpha x + y) * gain, the norm after the residual sum, in place; the same pass writes the next sublayer's
@@ -295,7 +300,7 @@ __global__ void token_shift_kernel(const float* __restrict__ h, long long ldh, c
   st32(out + (long long)r * ldo + c, fmaf(prev - cur, mu[c], cur));
 }
 
-// Short causal convolution added to its input.  A thread owns V channels of one TILE of consecutive rows of a request and walks the
+// Short causal convolution, added to its input or by itself.  A thread owns V channels of one TILE of consecutive rows of a request and walks the
 // rows with the K - 1 inputs before them in registers.  Tiles (and full chunks) are at least K - 1 rows long, so only the thread of a
 // request's FIRST tile reaches back past the rows of this step into the request's slot: it reads the carried inputs and then stores
 // the request's last K - 1 inputs there, and no other thread of the launch touches them.  The slot holds K - 1 rows of D, oldest
@@ -304,7 +309,7 @@ template <typename OT, int V, int K>
 __global__ void causal_conv_kernel(const float* __restrict__ h, long long ldh, const float* __restrict__ w, int D, const int* __restrict__ chunk_seq,
                                    const int* __restrict__ chunk_row0, const int* __restrict__ chunk_len, int subs, int tile,
                                    const int* __restrict__ row_pos, const int* __restrict__ seq_row0, const int* __restrict__ seq_slot,
-                                   float* __restrict__ state, long long slot_stride, OT* __restrict__ out, long long ldo) {
+                                   float* __restrict__ state, long long slot_stride, OT* __restrict__ out, long long ldo, float own) {
   const int ck = blockIdx.x / subs, sub = blockIdx.x % subs;
   const int c = (blockIdx.y * blockDim.x + threadIdx.x) * V;
   if (sub * tile >= chunk_len[ck] || c >= D) return;
@@ -337,7 +342,9 @@ __global__ void causal_conv_kernel(const float* __restrict__ h, long long ldh, c
   for (int t = 0; t < rows; ++t) {
     const long long r = r0 + t;
     win[K - 1] = ldv<V>(h + r * ldh + c);
-    f32vec<V> y = win[K - 1];
+    f32vec<V> y;
+#pragma unroll
+    for (int i = 0; i < V; ++i) y.v[i] = own * win[K - 1].v[i];
 #pragma unroll
     for (int k = 0; k < K; ++k)
 #pragma unroll
@@ -354,7 +361,7 @@ template <typename OT>
 __global__ void causal_conv_long_kernel(const float* __restrict__ h, long long ldh, const float* __restrict__ w, int K, int D,
                                         const int* __restrict__ chunk_seq, const int* __restrict__ chunk_row0, const int* __restrict__ chunk_len,
                                         const int* __restrict__ row_pos, const int* __restrict__ seq_row0, const int* __restrict__ seq_slot,
-                                        float* state, long long slot_stride, OT* __restrict__ out, long long ldo) {
+                                        float* state, long long slot_stride, OT* __restrict__ out, long long ldo, float own) {
   const int ck = blockIdx.x, c = blockIdx.y * blockDim.x + threadIdx.x;
   if (c >= D) return;
   const int s = chunk_seq[ck], first = seq_row0[s], end = seq_row0[s + 1], r0 = chunk_row0[ck];
@@ -365,7 +372,7 @@ __global__ void causal_conv_long_kernel(const float* __restrict__ h, long long l
     return started ? slot[(long long)(K - 1 + r - first) * D] : 0.f;
   };
   for (int r = r0; r < r0 + chunk_len[ck]; ++r) {
-    float y = h[(long long)r * ldh + c];
+    float y = own * h[(long long)r * ldh + c];
     for (int k = 0; k < K; ++k) y = fmaf(w[(long long)k * D + c], input(r - (K - 1) + k), y);
     st32(out + (long long)r * ldo + c, y);
   }
@@ -382,6 +389,7 @@ struct ConvLaunch {
   const int *row_pos, *seq_row0, *seq_slot;
   float* state; long long slot_stride;
   void* out; long long ldo;
+  float own;      // 1: the convolution is added to its input, 0: it stands alone
 };
 
 template <typename OT, int V, int K>
@@ -391,7 +399,7 @@ static void launch_conv(const ConvLaunch& a, cudaStream_t stream) {
   const dim3 grid(a.n_chunks * subs, (cols + threads - 1) / threads);
   causal_conv_kernel<OT, V, K><<<grid, threads, 0, stream>>>(a.h, a.ldh, a.w, a.D, a.chunk_seq, a.chunk_row0, a.chunk_len, subs, CONV_TILE,
                                                                  a.row_pos, a.seq_row0, a.seq_slot, a.state, a.slot_stride,
-                                                                 reinterpret_cast<OT*>(a.out), a.ldo);
+                                                                 reinterpret_cast<OT*>(a.out), a.ldo, a.own);
 }
 
 template <typename OT, int V>
@@ -408,7 +416,7 @@ static void launch_conv_taps(const ConvLaunch& a, int taps, cudaStream_t stream)
     default:
       causal_conv_long_kernel<OT><<<dim3(a.n_chunks, (a.D + CONV_THREADS - 1) / CONV_THREADS), CONV_THREADS, 0, stream>>>(
           a.h, a.ldh, a.w, taps, a.D, a.chunk_seq, a.chunk_row0, a.chunk_len, a.row_pos, a.seq_row0, a.seq_slot, a.state, a.slot_stride,
-          reinterpret_cast<OT*>(a.out), a.ldo);
+          reinterpret_cast<OT*>(a.out), a.ldo, a.own);
       break;
   }
 }
@@ -498,13 +506,268 @@ post_norm_kernel(float* __restrict__ x, long long ldx, const float* __restrict__
   for (int c = tid * V + POST_KEEP * step; c < D; c += step) finish(c, ldv<V>(xr + c));
 }
 
+// The embedding with learned positions, written `copies` times side by side (row stride ldo >= copies * D)
+__global__ void embed_streams_kernel(const int* __restrict__ ids, int R, const bf16* __restrict__ table, long long ldt, int vocab, float scale,
+                                     const bf16* __restrict__ pos_table, long long ldp, int n_pos, const int* __restrict__ row_pos,
+                                     float* __restrict__ out, long long ldo, int D, int copies) {
+  const int r = blockIdx.x;
+  if (r >= R) return;
+  int id = ids[r];
+  if (id < 0 || id >= vocab) id = 0;   // the host validates ids and positions; this only keeps a bad one inside the tables
+  const bf16* src = table + (long long)id * ldt;
+  const bf16* pv = nullptr;
+  if (pos_table != nullptr) {
+    const int p = row_pos[r];
+    pv = pos_table + (long long)(p < n_pos ? p : n_pos - 1) * ldp;
+  }
+  float* dst = out + (long long)r * ldo;
+  for (int c = threadIdx.x; c < D; c += blockDim.x) {
+    const float v = fmaf(__bfloat162float(src[c]), scale, pv != nullptr ? __bfloat162float(pv[c]) : 0.f);
+    for (int s = 0; s < copies; ++s) dst[(long long)s * D + c] = v;
+  }
+}
+
+// Token shift with n mixing vectors.  One thread per (row, V channels); the slot is touched by the thread of a request's first row only,
+// as in token_shift_kernel.
+template <typename OT, int V>
+__global__ void token_shift_mix_kernel(const float* __restrict__ h, long long ldh, const float* __restrict__ mu, int n, int R, int D,
+                                       const int* __restrict__ row_seq, const int* __restrict__ row_pos, const int* __restrict__ seq_row0,
+                                       const int* __restrict__ seq_slot, float* __restrict__ state, long long slot_stride,
+                                       OT* __restrict__ out, long long ldo, long long mix_stride) {
+  const int DV = D / V;
+  const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= (long long)R * DV) return;
+  const int r = (int)(i / DV), c = (int)(i % DV) * V;
+  const int s = row_seq[r];
+  const f32vec<V> cur = ldv<V>(h + (long long)r * ldh + c);
+  f32vec<V> step;
+#pragma unroll
+  for (int k = 0; k < V; ++k) step.v[k] = 0.f;
+  if (r == seq_row0[s]) {
+    float* slot = state + (long long)seq_slot[s] * slot_stride + c;
+    if (row_pos[r] > 0) step = ldv<V>(slot);
+    stv<V>(slot, ldv<V>(h + (long long)(seq_row0[s + 1] - 1) * ldh + c));
+  } else {
+    step = ldv<V>(h + (long long)(r - 1) * ldh + c);
+  }
+#pragma unroll
+  for (int k = 0; k < V; ++k) step.v[k] -= cur.v[k];
+  for (int m = 0; m < n; ++m) {
+    const f32vec<V> w = ldv<V>(mu + (long long)m * D + c);
+    f32vec<V> y;
+#pragma unroll
+    for (int k = 0; k < V; ++k) y.v[k] = fmaf(step.v[k], w.v[k], cur.v[k]);
+    stv<V>(out + m * mix_stride + (long long)r * ldo + c, y);
+  }
+}
+
+// Hyper-connections: one CTA per row.  The row's copies x_0 .. x_(n-1) lie side by side.  With y the sublayer before is closed (every copy
+// from the old ones), with gain the next one is opened: u = sum_s in[s] x_s is kept in registers for the first HYPER_KEEP column groups of
+// a thread (and made again from the copies beyond them) while the row's mean square is summed.  S: the number of copies, 0: any number
+// up to HYPER_MAX.  With mu (one-token steps: row m is the only row of request m) the operands are h + (h' - h) * mu_i, h' the row
+// carried in the request's slot (zeros at position 0), and the slot then takes h; a thread reads and writes its own columns only.
+constexpr int HYPER_THREADS = 256, HYPER_KEEP = 4, HYPER_MAX = 32;
+struct HyperArgs {
+  float* x; long long ldx; int n, D;
+  const float* y; long long ldy; const float* mix; const float* out_w;
+  const float* in_w; const float* gain; float eps;
+  void* h; long long ldh;
+  const float* mu; int n_mix; long long mix_stride;
+  const int* row_pos; const int* row_slot; float* state; long long slot_stride;
+};
+template <typename OT, int V, int S>
+__global__ void __launch_bounds__(HYPER_THREADS)
+hyper_kernel(HyperArgs a) {
+  constexpr int CAP = S > 0 ? S : HYPER_MAX;
+  __shared__ float mix_s[CAP * CAP], out_s[CAP], in_s[CAP], red[HYPER_THREADS / 32];
+  const int n = S > 0 ? S : a.n;
+  const long long m = blockIdx.x;
+  const int tid = threadIdx.x, step = blockDim.x * V, D = a.D;
+  for (int i = tid; i < n * n; i += blockDim.x) mix_s[i] = a.y != nullptr ? a.mix[i] : 0.f;
+  for (int i = tid; i < n; i += blockDim.x) {
+    out_s[i] = a.y != nullptr ? a.out_w[i] : 0.f;
+    in_s[i] = a.gain != nullptr ? (a.in_w != nullptr ? a.in_w[i] : 1.f) : 0.f;
+  }
+  __syncthreads();
+  float* xr = a.x + m * a.ldx;
+  const float* yr = a.y != nullptr ? a.y + m * a.ldy : nullptr;
+  f32vec<V> keep[HYPER_KEEP];
+  float ss = 0.f;
+  auto advance = [&](int c) {      // columns c .. c + V - 1: close, and the sum the next sublayer reads
+    f32vec<V> x[CAP], u;
+#pragma unroll
+    for (int s = 0; s < n; ++s) x[s] = ldv<V>(xr + (long long)s * D + c);
+#pragma unroll
+    for (int i = 0; i < V; ++i) u.v[i] = 0.f;
+    if (yr != nullptr) {
+      const f32vec<V> yv = ldv<V>(yr + c);
+#pragma unroll
+      for (int t = 0; t < n; ++t) {
+        f32vec<V> z;
+#pragma unroll
+        for (int i = 0; i < V; ++i) z.v[i] = out_s[t] * yv.v[i];
+#pragma unroll
+        for (int s = 0; s < n; ++s)
+#pragma unroll
+          for (int i = 0; i < V; ++i) z.v[i] = fmaf(mix_s[s * n + t], x[s].v[i], z.v[i]);
+        stv<V>(xr + (long long)t * D + c, z);
+#pragma unroll
+        for (int i = 0; i < V; ++i) u.v[i] = fmaf(in_s[t], z.v[i], u.v[i]);
+      }
+    } else {
+#pragma unroll
+      for (int s = 0; s < n; ++s)
+#pragma unroll
+        for (int i = 0; i < V; ++i) u.v[i] = fmaf(in_s[s], x[s].v[i], u.v[i]);
+    }
+#pragma unroll
+    for (int i = 0; i < V; ++i) ss = fmaf(u.v[i], u.v[i], ss);
+    return u;
+  };
+#pragma unroll
+  for (int it = 0; it < HYPER_KEEP; ++it) {
+    const int c = tid * V + it * step;
+    if (c < D) keep[it] = advance(c);
+  }
+  for (int c = tid * V + HYPER_KEEP * step; c < D; c += step) advance(c);
+  if (a.gain == nullptr) return;
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+  if ((tid & 31) == 0) red[tid >> 5] = ss;
+  __syncthreads();
+  float total = 0.f;
+  for (int k = 0; k < (int)(blockDim.x >> 5); ++k) total += red[k];
+  const float r = 1.0f / sqrtf(total / (float)D + a.eps);
+  float* slot = a.mu != nullptr ? a.state + (long long)a.row_slot[m] * a.slot_stride : nullptr;
+  const bool started = a.mu != nullptr && a.row_pos[m] > 0;
+  OT* hr = reinterpret_cast<OT*>(a.h) + m * a.ldh;
+  auto finish = [&](int c, f32vec<V> u) {
+    const f32vec<V> g = ldv<V>(a.gain + c);
+#pragma unroll
+    for (int i = 0; i < V; ++i) u.v[i] = u.v[i] * r * g.v[i];
+    if (a.mu == nullptr) {
+      stv<V>(hr + c, u);
+      return;
+    }
+    f32vec<V> prev;
+#pragma unroll
+    for (int i = 0; i < V; ++i) prev.v[i] = 0.f;
+    if (started) prev = ldv<V>(slot + c);
+    stv<V>(slot + c, u);
+    for (int k = 0; k < a.n_mix; ++k) {
+      const f32vec<V> w = ldv<V>(a.mu + (long long)k * D + c);
+      f32vec<V> o;
+#pragma unroll
+      for (int i = 0; i < V; ++i) o.v[i] = fmaf(prev.v[i] - u.v[i], w.v[i], u.v[i]);
+      stv<V>(hr + k * a.mix_stride + c, o);
+    }
+  };
+#pragma unroll
+  for (int it = 0; it < HYPER_KEEP; ++it) {
+    const int c = tid * V + it * step;
+    if (c < D) finish(c, keep[it]);
+  }
+  for (int c = tid * V + HYPER_KEEP * step; c < D; c += step) {
+    f32vec<V> u;
+#pragma unroll
+    for (int i = 0; i < V; ++i) u.v[i] = 0.f;
+    for (int s = 0; s < n; ++s) {
+      const f32vec<V> x = ldv<V>(xr + (long long)s * D + c);
+#pragma unroll
+      for (int i = 0; i < V; ++i) u.v[i] = fmaf(in_s[s], x.v[i], u.v[i]);
+    }
+    finish(c, u);
+  }
+}
+
+template <typename OT, int V>
+static void launch_hyper(const HyperArgs& a, int M, int threads, cudaStream_t stream) {
+  switch (a.n) {
+    case 1: hyper_kernel<OT, V, 1><<<M, threads, 0, stream>>>(a); break;
+    case 2: hyper_kernel<OT, V, 2><<<M, threads, 0, stream>>>(a); break;
+    case 3: hyper_kernel<OT, V, 3><<<M, threads, 0, stream>>>(a); break;
+    case 4: hyper_kernel<OT, V, 4><<<M, threads, 0, stream>>>(a); break;
+    default: hyper_kernel<OT, V, 0><<<M, threads, 0, stream>>>(a); break;
+  }
+}
+
 }  // namespace lp
 
 using namespace lp;
 
+extern "C" int lp_embed_streams_f32(const int* ids, int R, const void* table, long long ldt, int vocab, float scale, const void* pos_table,
+                                    long long ldp, int n_pos, const int* row_pos, float* out, long long ldo, int D, int copies, void* stream_) {
+  cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
+  LP_REQUIRE(ids != nullptr && table != nullptr && out != nullptr && R >= 0 && D > 0 && vocab > 0 && copies > 0 && ldo >= (long long)copies * D,
+             "lp_embed_streams_f32: bad arguments");
+  LP_REQUIRE(pos_table == nullptr || (n_pos > 0 && row_pos != nullptr), "lp_embed_streams_f32: a position table without positions");
+  if (R == 0) return 0;
+  embed_streams_kernel<<<R, 128, 0, stream>>>(ids, R, reinterpret_cast<const bf16*>(table), ldt, vocab, scale,
+                                              reinterpret_cast<const bf16*>(pos_table), ldp, n_pos, row_pos, out, ldo, D, copies);
+  note_launch();
+  LP_CHECK_CUDA(cudaGetLastError());
+  return 0;
+}
+
+extern "C" int lp_token_shift_mix_f32(const float* h, long long ldh, const float* mu, int n, int R, int D, const int* row_seq,
+                                      const int* row_pos, const int* seq_row0, const int* seq_slot, float* state, long long slot_stride,
+                                      void* out, long long ldo, long long mix_stride, int out_fp32, void* stream_) {
+  cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
+  LP_REQUIRE(h != nullptr && mu != nullptr && out != nullptr && state != nullptr && row_seq != nullptr && row_pos != nullptr &&
+                 seq_row0 != nullptr && seq_slot != nullptr && n > 0 && R >= 0 && D > 0 && slot_stride >= D,
+             "lp_token_shift_mix_f32: bad arguments");
+  LP_REQUIRE(h != out, "lp_token_shift_mix_f32: a row reads its neighbour as it came in, so it cannot run in place");
+  if (R == 0) return 0;
+  const bool v4 = vec4_ok(D, {h, mu, state, out}, {ldh, slot_stride, ldo, mix_stride});
+  const unsigned grid = (unsigned)(((long long)R * (v4 ? D / 4 : D) + 255) / 256);
+  if (out_fp32 && v4)
+    token_shift_mix_kernel<float, 4><<<grid, 256, 0, stream>>>(h, ldh, mu, n, R, D, row_seq, row_pos, seq_row0, seq_slot, state, slot_stride,
+                                                               reinterpret_cast<float*>(out), ldo, mix_stride);
+  else if (out_fp32)
+    token_shift_mix_kernel<float, 1><<<grid, 256, 0, stream>>>(h, ldh, mu, n, R, D, row_seq, row_pos, seq_row0, seq_slot, state, slot_stride,
+                                                               reinterpret_cast<float*>(out), ldo, mix_stride);
+  else if (v4)
+    token_shift_mix_kernel<bf16, 4><<<grid, 256, 0, stream>>>(h, ldh, mu, n, R, D, row_seq, row_pos, seq_row0, seq_slot, state, slot_stride,
+                                                              reinterpret_cast<bf16*>(out), ldo, mix_stride);
+  else
+    token_shift_mix_kernel<bf16, 1><<<grid, 256, 0, stream>>>(h, ldh, mu, n, R, D, row_seq, row_pos, seq_row0, seq_slot, state, slot_stride,
+                                                              reinterpret_cast<bf16*>(out), ldo, mix_stride);
+  note_launch();
+  LP_CHECK_CUDA(cudaGetLastError());
+  return 0;
+}
+
+extern "C" int lp_hyper_max_streams(void) { return HYPER_MAX; }
+
+extern "C" int lp_hyper_f32(const lp_hyper_desc* d, int M, void* stream_) {
+  cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
+  LP_REQUIRE(d != nullptr && d->x != nullptr && d->n >= 1 && d->n <= HYPER_MAX && d->D > 0 && M >= 0 && d->ldx >= (long long)d->n * d->D,
+             "lp_hyper_f32: bad arguments (1 .. %d streams)", HYPER_MAX);
+  LP_REQUIRE(d->y == nullptr || (d->mix != nullptr && d->out_w != nullptr), "lp_hyper_f32: a result without its connection weights");
+  LP_REQUIRE((d->gain != nullptr) == (d->h != nullptr) && (d->y != nullptr || d->gain != nullptr), "lp_hyper_f32: nothing to do");
+  LP_REQUIRE(d->mu == nullptr || (d->gain != nullptr && d->n_mix > 0 && d->row_pos != nullptr && d->row_slot != nullptr && d->state != nullptr &&
+                                  d->slot_stride >= d->D),
+             "lp_hyper_f32: a token shift without its slot");
+  if (M == 0) return 0;
+  HyperArgs a{d->x, d->ldx, d->n, d->D, d->y, d->ldy, d->mix, d->out_w, d->in_w, d->gain, d->eps, d->h, d->ldh, d->mu, d->n_mix,
+              d->mix_stride, d->row_pos, d->row_slot, d->state, d->slot_stride};
+  const bool v4 = vec4_ok(d->D, {d->x, d->y, d->gain, d->h, d->mu, d->state},
+                          {d->ldx, d->y != nullptr ? d->ldy : 0, d->h != nullptr ? d->ldh : 0, d->mu != nullptr ? d->mix_stride : 0,
+                           d->state != nullptr ? d->slot_stride : 0});
+  int threads = v4 ? d->D / 4 : d->D;
+  threads = threads >= HYPER_THREADS ? HYPER_THREADS : (threads + 31) / 32 * 32;
+  if (d->h_fp32 && v4) launch_hyper<float, 4>(a, M, threads, stream);
+  else if (d->h_fp32) launch_hyper<float, 1>(a, M, threads, stream);
+  else if (v4) launch_hyper<bf16, 4>(a, M, threads, stream);
+  else launch_hyper<bf16, 1>(a, M, threads, stream);
+  note_launch();
+  LP_CHECK_CUDA(cudaGetLastError());
+  return 0;
+}
+
 extern "C" int lp_causal_conv_max_taps(void) { return CONV_MAX_TAPS; }
 
-extern "C" int lp_causal_conv_f32(const float* h, long long ldh, const float* w, int taps, int D, int n_chunks, const int* chunk_seq,
+extern "C" int lp_causal_conv_f32(const float* h, long long ldh, const float* w, int taps, int add_input, int D, int n_chunks, const int* chunk_seq,
                                   const int* chunk_row0, const int* chunk_len, int longest_chunk, const int* row_pos, const int* seq_row0,
                                   const int* seq_slot, float* state, long long slot_stride, void* out, long long ldo, int out_fp32,
                                   void* stream_) {
@@ -517,7 +780,8 @@ extern "C" int lp_causal_conv_f32(const float* h, long long ldh, const float* w,
   LP_REQUIRE(longest_chunk >= 1 && longest_chunk <= LP_RETENTION_CHUNK, "lp_causal_conv_f32: longest_chunk=%d", longest_chunk);
   LP_REQUIRE(h != out, "lp_causal_conv_f32: a row reads its neighbours as they came in, so it cannot run in place");
   if (n_chunks == 0) return 0;
-  const ConvLaunch a{h, ldh, w, D, n_chunks, chunk_seq, chunk_row0, chunk_len, longest_chunk, row_pos, seq_row0, seq_slot, state, slot_stride, out, ldo};
+  const ConvLaunch a{h, ldh, w, D, n_chunks, chunk_seq, chunk_row0, chunk_len, longest_chunk, row_pos, seq_row0, seq_slot, state, slot_stride, out, ldo,
+                     add_input ? 1.f : 0.f};
   const bool v4 = taps <= CONV_WINDOW_TAPS && vec4_ok(D, {h, w, state, out}, {ldh, ldo, taps > 1 ? slot_stride : 0});
   if (out_fp32 && v4) launch_conv_taps<float, 4>(a, taps, stream);
   else if (out_fp32) launch_conv_taps<float, 1>(a, taps, stream);

@@ -5,11 +5,15 @@
 //   visibility   window (tokens j with 0 <= i - j < window), keep_first (the request's first tokens stay visible), pool (every block
 //                of P tokens that lies wholly before the window is seen as ONE key / value, the mean of its cached rows)
 //   scores       scale, softcap * tanh(score / softcap), sink (softmax denominator + 1), a distance bias per head: after the cap
-//                dist_amp[h] * ln(1 + dist_rate[h] * (i - j)) is taken off
+//                dist_amp[h] * ln(1 + dist_rate[h] * (i - j)), or dist_amp[h] * (i - j), is taken off
 //   projections  RMS norm of q and k per head or over the whole projection, a temperature per query head (q_temp), rotation of the first rot_dims dimensions of q and k,
 //                optional rotation of the values by their own position with the head output turned back by the query's position
 //                (the weighted sum then depends on the distances i - j only)
 //
+//                a query temperature that grows with the logarithm of the position; the values may be the keys themselves (v_is_k: one
+//                cached row serves both); q and k may pass a short causal convolution first (one-token steps: here; prompts: by
+//                lp_causal_conv_f32 before)
+//   output       an elementwise gate sigmoid(gate) and a constant factor on the way out
 //   mixing       talk: the softmax weights of the heads are mixed before they meet the values, weight_h <- sum_g talk[h, g] weight_g;
 //                an output gate sigmoid(g) taken from the fused projection multiplies the heads' outputs
 //
@@ -49,22 +53,34 @@ struct WinArgs {
   const float* talk; int g_off;
   int chunk, kv_shared;
   const float* q_temp; const float* dist_amp; const float* dist_rate;
+  int roww, v_base;      // floats per cache row, and where its values start (v_is_k: at the keys)
+  int v_is_k;
+  const float* gate; long long ldg; float out_scale;
+  float pos_temp_coef; int pos_temp_every;
+  const float* conv_w; int conv_taps; const int* row_slot; float* conv_state; long long conv_stride;
 };
 
 __device__ __forceinline__ float* win_token_row(const WinArgs& a, int seq, int pos) {
   const int page = a.page_table[(long long)seq * a.max_pages + pos / a.page_size];
-  return a.cache + ((long long)page * a.page_size + pos % a.page_size) * (long long)(a.kv_heads * (a.dim + a.vdim));
+  return a.cache + ((long long)page * a.page_size + pos % a.page_size) * (long long)a.roww;
 }
 __device__ __forceinline__ float* win_block_row(const WinArgs& a, int seq, int block) {
   const int page = a.pooled_table[(long long)seq * a.max_pooled_pages + block / a.page_size];
-  return a.pooled + ((long long)page * a.page_size + block % a.page_size) * (long long)(a.kv_heads * (a.dim + a.vdim));
+  return a.pooled + ((long long)page * a.page_size + block % a.page_size) * (long long)a.roww;
 }
 
-// what is taken off a score at distance d >= 0: amp ln(1 + rate d).  `exact`: the accurate logarithm (fp32 results); else the fast
+// what is taken off a score at distance d >= 0: amp d, or amp ln(1 + rate d).  `exact`: the accurate logarithm (fp32 results); else the fast
 // one, whose absolute error of a few 1e-7 is far below the rounding of a 16-bit output.
-__device__ __forceinline__ float win_distance_bias(float amp, float rate, int d, bool exact) {
+__device__ __forceinline__ float win_distance_bias(bool linear, float amp, float rate, int d, bool exact) {
+  if (linear) return amp * (float)d;
   const float x = fmaf(rate, (float)(d > 0 ? d : 0), 1.0f);
   return amp * (exact ? logf(x) : __logf(x));
+}
+
+// column c of row r on its way out: gate and factor
+__device__ __forceinline__ float win_out(const WinArgs& a, int r, int c, float v) {
+  if (a.gate != nullptr) v /= 1.0f + expf(-a.gate[(long long)r * a.ldg + c]);
+  return v * a.out_scale;
 }
 
 // the two members of rotation pair i
@@ -110,6 +126,23 @@ window_attn_prep_kernel(WinArgs a, int R, const int* __restrict__ row_seq, const
   float* x = a.qkv + (long long)r * a.ld;
   const int kvh = a.kv_shared ? 0 : a.kv_heads;      // key / value heads this row brings (none: they are another layer's)
   const int units = a.heads + kvh;
+  if (a.conv_w != nullptr) {      // the row is its request's only one: a thread owns its channels of the row and of the slot
+    const int C = (a.heads + a.kv_heads) * a.dim, K = a.conv_taps;
+    float* slot = K > 1 ? a.conv_state + (long long)a.row_slot[r] * a.conv_stride : nullptr;
+    for (int c = tid; c < C; c += blockDim.x) {
+      const float cur = x[a.q_off + c];
+      float y = 0.f;
+      for (int k = 0; k < K - 1; ++k) {
+        const float old = pos > 0 ? slot[(long long)k * C + c] : 0.f;
+        y = fmaf(a.conv_w[(long long)k * C + c], old, y);
+        if (k > 0) slot[(long long)(k - 1) * C + c] = old;
+      }
+      if (K > 1) slot[(long long)(K - 2) * C + c] = cur;
+      x[a.q_off + c] = fmaf(a.conv_w[(long long)(K - 1) * C + c], cur, y);
+    }
+    __syncthreads();
+  }
+  const float pos_temp = a.pos_temp_every > 0 ? fmaf(a.pos_temp_coef, logf((float)((pos + 1) / a.pos_temp_every) + 1.0f), 1.0f) : 1.0f;
   // biases of the projections: added in place before anything reads the row
   if (a.q_bias != nullptr || a.k_bias != nullptr || a.v_bias != nullptr) {
     if (a.q_bias != nullptr)
@@ -173,6 +206,7 @@ window_attn_prep_kernel(WinArgs a, int R, const int* __restrict__ row_seq, const
       gain = (is_q ? a.q_gain : a.k_gain) + hl * a.dim;
     }
     if (is_q && a.q_temp != nullptr) rinv *= a.q_temp[hl];      // the head's temperature scales its query
+    if (is_q) rinv *= pos_temp;
     if (e < half) {
       int d0, d1;
       win_pair(a.rot_layout, half, e, d0, d1);
@@ -198,10 +232,11 @@ window_attn_prep_kernel(WinArgs a, int R, const int* __restrict__ row_seq, const
   const int vhalf = a.v_inv_freq != nullptr ? a.v_rot_dims >> 1 : 0;
   const int vrot = 2 * vhalf;
   const int vper = a.vdim - vhalf;
+  if (a.v_is_k) return;
   for (int it = tid; it < kvh * vper; it += blockDim.x) {
     const int g = it / vper, e = it % vper;
     const float* src = x + a.v_off + g * a.vdim;
-    float* dst = crow + a.kv_heads * a.dim + g * a.vdim;
+    float* dst = crow + a.v_base + g * a.vdim;
     const float vinv = a.v_norm ? 1.0f / sqrtf(s_vss[g] / (float)a.vdim + a.eps) : 1.f;      // unit RMS per value head, cached so
     if (e < vhalf) {
       int d0, d1;
@@ -226,7 +261,7 @@ window_attn_pool_kernel(WinArgs a, int n_seqs, const int* __restrict__ seq_row0,
   const int pos0 = seq_pos0[s], len = seq_row0[s + 1] - seq_row0[s];
   const int b = pos0 / a.pool + blockIdx.y;
   if (b >= (pos0 + len) / a.pool) return;      // block b is complete when its last token b P + P - 1 has been written
-  const int roww = a.kv_heads * (a.dim + a.vdim);
+  const int roww = a.roww;
   const int c = blockIdx.z * WIN_POOL_THREADS + threadIdx.x;      // one column of the row per thread, the rows in their order
   if (c >= roww) return;
   float sum = 0.f;
@@ -256,14 +291,14 @@ window_attn_kernel(WinArgs a, int R, const int* __restrict__ row_seq, const int*
   for (int i = tid; i < QH * a.dim; i += blockDim.x) q_s[i] = q[i];
   __syncthreads();
   const WinVisible vis = win_visible(a, pos);
-  const int v_off = a.kv_heads * a.dim + g * a.vdim;
+  const int v_off = a.v_base + g * a.vdim;
   const bool vec = (a.dim % 4 == 0) && (a.vdim % 4 == 0);      // rows and head offsets are then 16-byte aligned
   const bool quads = vec && (a.dim % 16 == 0);
   float mx[QH], den[QH], acc[QH][NV], amp[QH], rate[QH];
 #pragma unroll
   for (int h = 0; h < QH; ++h) {
     amp[h] = DIST ? a.dist_amp[h0 + h] : 0.f;
-    rate[h] = DIST ? a.dist_rate[h0 + h] : 0.f;
+    rate[h] = DIST && a.dist_rate != nullptr ? a.dist_rate[h0 + h] : 0.f;
     // the sink is a key of score 0 without a value: warp 0 starts from it
     mx[h] = (a.sink && warp == 0) ? 0.f : -INFINITY;
     den[h] = (a.sink && warp == 0) ? 1.f : 0.f;
@@ -345,7 +380,7 @@ window_attn_kernel(WinArgs a, int R, const int* __restrict__ row_seq, const int*
     for (int h = 0; h < QH; ++h) {
       float s = sc[h] * a.scale;
       if (a.softcap > 0.f) s = a.softcap * tanhf(s / a.softcap);
-      if (DIST) s -= win_distance_bias(amp[h], rate[h], dist, out_fp32);
+      if (DIST) s -= win_distance_bias(a.dist_rate == nullptr, amp[h], rate[h], dist, out_fp32);
       if (!valid) s = -INFINITY;
       float top = s;
 #pragma unroll
@@ -434,6 +469,7 @@ window_attn_kernel(WinArgs a, int R, const int* __restrict__ row_seq, const int*
       // rotation by the negative angle: (u, v) -> (u cos + v sin, v cos - u sin)
       v = first ? o[c] * cs + o[partner] * s : o[c] * cs - o[partner] * s;
     }
+    v = win_out(a, r, (h0 + h) * a.vdim + c, v);
     const long long at = (long long)r * ldo + (long long)(h0 + h) * a.vdim + c;
     if (out_fp32) reinterpret_cast<float*>(out)[at] = v;
     else reinterpret_cast<bf16*>(out)[at] = __float2bfloat16(v);
@@ -489,13 +525,13 @@ window_attn_tile_kernel(WinArgs a, int n_chunks, const int* __restrict__ chunk_s
   uni.n_blocks = last.n_blocks;
   uni.lo = r_lo[0];
   uni.count = uni.n_keep + uni.n_blocks + (pos0 + nrows - 1 - uni.lo + 1);
-  const int v_off = a.kv_heads * a.dim + g * a.vdim;
+  const int v_off = a.v_base + g * a.vdim;
   const bool quads = (a.dim % 16 == 0) && (a.vdim % 4 == 0);
   float mx[X], den[X], acc[X][NV], amp[QH], rate[QH];
 #pragma unroll
   for (int h = 0; h < QH; ++h) {
     amp[h] = DIST ? a.dist_amp[h0 + h] : 0.f;
-    rate[h] = DIST ? a.dist_rate[h0 + h] : 0.f;
+    rate[h] = DIST && a.dist_rate != nullptr ? a.dist_rate[h0 + h] : 0.f;
   }
 #pragma unroll
   for (int x = 0; x < X; ++x) {
@@ -586,7 +622,7 @@ window_attn_tile_kernel(WinArgs a, int n_chunks, const int* __restrict__ chunk_s
       else seen = seen && idx >= r_lo[rq] && idx <= pos0 + rq;
       float s = sc[x] * a.scale;
       if (a.softcap > 0.f) s = a.softcap * tanhf(s / a.softcap);
-      if (DIST) s -= win_distance_bias(amp[x % QH], rate[x % QH], pos0 + rq - idx, out_fp32);
+      if (DIST) s -= win_distance_bias(a.dist_rate == nullptr, amp[x % QH], rate[x % QH], pos0 + rq - idx, out_fp32);
       if (!seen) s = -INFINITY;
       float top = s;
 #pragma unroll
@@ -681,6 +717,7 @@ window_attn_tile_kernel(WinArgs a, int n_chunks, const int* __restrict__ chunk_s
       sincosf((float)(pos0 + rq) * a.v_inv_freq[pair], &sn, &cs);
       v = first ? o[cc] * cs + o[partner] * sn : o[cc] * cs - o[partner] * sn;
     }
+    v = win_out(a, r0 + rq, (h0 + h) * a.vdim + cc, v);
     const long long at = (long long)(r0 + rq) * ldo + (long long)(h0 + h) * a.vdim + cc;
     if (out_fp32) reinterpret_cast<float*>(out)[at] = v;
     else reinterpret_cast<bf16*>(out)[at] = __float2bfloat16(v);
@@ -889,7 +926,7 @@ window_attn_talk_kernel(WinArgs a, int R, const int* __restrict__ row_seq, const
       for (int x = 0; x < QH; ++x) acc[i][rq][x] = 0.f;
   const int nqg = ratio / QH;                       // query-head groups per key / value head
   const int units = a.kv_heads * nqg * a.vdim;      // (key / value head, query group, channel)
-  const int v_base = a.kv_heads * a.dim;
+  const int v_base = a.v_base;
   for (int t0 = 0; t0 < count; t0 += tile) {
     const int cnt = count - t0 < tile ? count - t0 : tile;
     talk_tile_scores<RQ>(a, tr, seq, t0, cnt, tile, hd4, q_s, p_s, row_s, m_s, l_s, true, tid, NT);
@@ -1085,8 +1122,23 @@ static int fill_win(WinArgs& a, const lp_window_attn_desc* d, bool need_q) {
   a.q_bias = d->q_bias; a.k_bias = d->k_bias; a.v_bias = d->v_bias; a.v_norm = d->v_norm;
   a.talk = d->talk; a.g_off = d->g_off;
   a.q_temp = d->q_temp; a.dist_amp = d->dist_amp; a.dist_rate = d->dist_rate;
-  LP_REQUIRE((d->dist_amp != nullptr) == (d->dist_rate != nullptr), "lp_window_attn: one half of a distance bias without the other");
+  LP_REQUIRE(d->dist_amp != nullptr || d->dist_rate == nullptr, "lp_window_attn: a distance rate without an amplitude");
   LP_REQUIRE(d->dist_amp == nullptr || d->pool == 0, "lp_window_attn: a distance bias to pooled blocks is not defined");
+  LP_REQUIRE(!d->v_is_k || (d->vdim == d->dim && d->v_bias == nullptr && !d->v_norm && d->v_inv_freq == nullptr),
+             "lp_window_attn: values that are the keys have the keys' size and nothing of their own");
+  a.v_is_k = d->v_is_k;
+  a.v_base = d->v_is_k ? 0 : d->kv_heads * d->dim;
+  a.roww = a.v_base + d->kv_heads * d->vdim;
+  a.gate = d->gate; a.ldg = d->ldg; a.out_scale = d->out_scale == 0.f ? 1.f : d->out_scale;
+  LP_REQUIRE(d->pos_temp_every >= 0, "lp_window_attn: pos_temp_every < 0");
+  a.pos_temp_coef = d->pos_temp_coef; a.pos_temp_every = d->pos_temp_every;
+  LP_REQUIRE(d->conv_w == nullptr || (d->conv_taps >= 1 && !d->kv_shared && d->k_off == d->q_off + d->heads * d->dim),
+             "lp_window_attn: a convolution over q and k needs them side by side");
+  LP_REQUIRE(d->conv_w == nullptr || d->conv_taps == 1 ||
+                 (d->row_slot != nullptr && d->conv_state != nullptr &&
+                  d->conv_stride >= (long long)(d->conv_taps - 1) * (d->heads + d->kv_heads) * d->dim),
+             "lp_window_attn: no room for the convolution's carried inputs");
+  a.conv_w = d->conv_w; a.conv_taps = d->conv_taps; a.row_slot = d->row_slot; a.conv_state = d->conv_state; a.conv_stride = d->conv_stride;
   return 0;
 }
 
@@ -1166,7 +1218,7 @@ extern "C" int lp_window_attn_pool(const lp_window_attn_desc* d, int n_seqs, con
   LP_REQUIRE(d->pool > 0 && seq_row0 != nullptr && seq_pos0 != nullptr, "lp_window_attn_pool: no pooled blocks in this description");
   if (n_seqs <= 0 || max_new_blocks <= 0) return 0;
   LP_REQUIRE(max_new_blocks <= 65535, "lp_window_attn_pool: %d blocks per request in one step", max_new_blocks);
-  const int roww = d->kv_heads * (d->dim + d->vdim);
+  const int roww = a.roww;
   window_attn_pool_kernel<<<dim3(n_seqs, max_new_blocks, (roww + WIN_POOL_THREADS - 1) / WIN_POOL_THREADS), WIN_POOL_THREADS, 0, stream>>>(
       a, n_seqs, seq_row0, seq_pos0);
   note_launch();

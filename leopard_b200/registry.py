@@ -65,6 +65,11 @@ def _komazen(path, **kw):
     return komazen.load(path, **kw)
 
 
+def _bezizen(path, **kw):
+    from . import bezizen
+    return bezizen.load(path, **kw)
+
+
 def _llava(path, **kw):
     from .hf import myLlavaForConditionalGeneration
     return myLlavaForConditionalGeneration.from_pretrained(path, **kw)
@@ -75,6 +80,7 @@ register("Ronelorn", _ronelorn)
 register("Gavatar", _gavatar)
 register("Kamosun", _kamosun)
 register("Komazen", _komazen)
+register("Bezizen", _bezizen)
 register("LlavaForConditionalGeneration", _llava)
 register("myLlavaForConditionalGeneration", _llava)
 register("llava", _llava)

@@ -1,8 +1,8 @@
 """Decoder-only language models described as a LIST OF LAYERS, on the 32-bit residual-stream kernels.
 
 A model is a `SeqLMConfig`: vocabulary, width, norm epsilon and style, and a tuple of `LayerConfig`s, each naming its sequence mixer
-(`RetentionConfig`, `LatentAttentionConfig`, `WindowAttentionConfig`, `MinGRUConfig`, `MLSTMConfig`, or a `ParallelMixerConfig` of
-two of them side by side) and its feed-forward
+(`RetentionConfig`, `LatentAttentionConfig`, `WindowAttentionConfig`, `MinGRUConfig`, `MLSTMConfig`, `WKVConfig`, `GatedLinearConfig`, or a
+`ParallelMixerConfig` of two of them side by side) and its feed-forward
 (`DenseFFConfig`, `MoEConfig` or none); a layer may run on another layer's weights with a cache or state of its own (a looped stack
 is such a list), shift its mixer's input towards the previous token's, run a short causal convolution over the input of its
 sublayers, and add a learned vector to the stream before it runs.  Every mechanism is a separate native entry point with its constants
@@ -32,6 +32,7 @@ from .seqcache import SequenceCache
 F32, BF16, I32 = torch.float32, torch.bfloat16, torch.int32
 TENSOR_CORE_MIN_ROWS = 64
 MOE_PAIRS_MAX = 64             # up to this many (token, choice) pairs the experts run as one-row weight-streaming problems
+PAD_PROJECTION_ROWS = 128      # a projection narrower than a tensor-core tile is padded with zero rows beside ones that are at least this wide
 MAX_DECODE_GRAPHS = 32         # captured decode layouts kept at a time
 PAGE_TABLE_STEP = 16           # decode batches round their page-table width up to a multiple of this
 
@@ -164,6 +165,12 @@ class WindowAttentionConfig:
     kv_from: Optional[int] = None
     head_temp: bool = False        # head h's scores are multiplied by mix.temp[h]
     distance_bias: bool = False    # mix.r1[h] * ln(1 + mix.r2[h] * (i - j)) is taken off head h's score (after the cap)
+    distance_slope: bool = False   # 2^(-8 (h + 1) / heads) * (i - j) is taken off head h's score (after the cap)
+    # > 0: q and k pass a causal convolution of that many taps over time on each channel right after their projection (mix.q.conv, mix.k.conv,
+    # [channels, taps]); the last taps - 1 projected values are part of the request's state, zeros before the first token
+    qk_conv: int = 0
+    values_are_keys: bool = False  # the keys as they leave the convolution are the values too (no mix.v; vdim = dim)
+    pos_temp: Optional[Tuple[float, int]] = None   # (coef, every): the query at position p is multiplied by 1 + coef ln(floor((p + 1) / every) + 1)
 
 
 @dataclass(frozen=True)
@@ -183,11 +190,36 @@ class MLSTMConfig:
 
 
 @dataclass(frozen=True)
+class WKVConfig:
+    """Time mixing over a matrix memory whose rows decay per key channel (csrc/lp_gla.cu).  With h' the previous token's input (part of the
+    request's state, zeros before the first token) the projections r, k, v, g and w each read a mix h + (h' - h) * mu of their own
+    (mix.mu.*); the decay is exp(-exp(mix.w2 tanh(mix.w1 .) + mix.w0)), the current token enters the read-out by its bonus mix.u instead of
+    through the state; every head's output is divided by its root mean square, then comes the gain mix.norm over the heads and silu(mix.g .)."""
+    heads: int
+    dim: int                       # key and value size
+
+
+@dataclass(frozen=True)
+class GatedLinearConfig:
+    """Gated linear attention on the same kernels: q scaled by dim^-1/2, a decay sigmoid(mix.a2 (mix.a1 h) + mix.a2.b)^(1 / tau) per key
+    channel, every head's output RMS-normed with a gain that the heads share (mix.norm [vdim]) and gated by silu(mix.g h)."""
+    heads: int
+    dim: int
+    vdim: int
+    tau: float
+
+
+AnyMixer = Union[RetentionConfig, LatentAttentionConfig, WindowAttentionConfig, MinGRUConfig, MLSTMConfig, WKVConfig, GatedLinearConfig]
+
+
+@dataclass(frozen=True)
 class ParallelMixerConfig:
     """Two mixers side by side on the same input (tensors under mix.left.* and mix.right.*); the result is half the sum of the two
-    outputs, each first RMS-normed over the model width with its own plain gain (mix.left.out, mix.right.out)."""
-    left: Union[RetentionConfig, LatentAttentionConfig, WindowAttentionConfig, MinGRUConfig, MLSTMConfig]
-    right: Union[RetentionConfig, LatentAttentionConfig, WindowAttentionConfig, MinGRUConfig, MLSTMConfig]
+    outputs, each first RMS-normed over the model width with its own plain gain (mix.left.out, mix.right.out) — or, with `scales`, simply
+    scales[0] * left + scales[1] * right (window attention beside gated linear attention)."""
+    left: AnyMixer
+    right: AnyMixer
+    scales: Optional[Tuple[float, float]] = None
 
 
 GLU_SLOPE = 1.702                  # the sigmoid's slope in the clamped gated unit
@@ -213,8 +245,11 @@ class MoEConfig:
     shared_ff: int = 0             # 0: no shared expert
     # "grouped_sigmoid": sigmoid scores, choice bias, best groups, weights = chosen scores / their sum;
     # "softmax_top": logits + mlp.router.b, the largest are chosen, weights = softmax over the chosen logits;
-    # "sigmoid_input": sigmoid scores, the largest are chosen, and a chosen expert runs on score * h (its output is not weighted)
+    # "sigmoid_input": sigmoid scores, the largest are chosen, and a chosen expert runs on score * h (its output is not weighted);
+    # "group_softmax": scores = softmax over all experts, a group counts by its largest score, only the best groups stay, weights = the
+    # chosen scores / their sum * weight_scale
     router: str = "grouped_sigmoid"
+    weight_scale: float = 1.0
     act: str = "silu_glu"          # the experts' unit: "silu_glu" (silu(gate) * up) or "clamp_glu" (DenseFFConfig) with the limits below
     limit: float = 0.0
     shared_limit: float = 0.0
@@ -223,7 +258,7 @@ class MoEConfig:
 
 @dataclass(frozen=True)
 class LayerConfig:
-    mixer: Union[RetentionConfig, LatentAttentionConfig, WindowAttentionConfig, MinGRUConfig, MLSTMConfig, ParallelMixerConfig]
+    mixer: Union[AnyMixer, ParallelMixerConfig]
     ff: Union[DenseFFConfig, MoEConfig, None]
     weights_of: Optional[int] = None   # run on that layer's tensors (mixer, feed-forward, norms); cache and state stay this layer's own
     # the mixer reads h_t + (h_(t-1) - h_t) * shift per channel instead of h_t (h: the normed stream; the previous token's h is part of
@@ -244,7 +279,7 @@ class SeqLMConfig:
     eps: float
     layers: Tuple[LayerConfig, ...]
     # "sandwich": x <- x + norm_b(sublayer(norm_a(x))), every norm with ONE gain; "pre": x <- x + residual_mult * sublayer(norm(x)),
-    # the norm's gain a vector stored around zero (x / rms * (1 + w)); "sandwich_vector": the sandwich form with such vector gains;
+    # the norm's gain a vector stored around zero (x / rms * (1 + w)); "pre_plain": the same with plain gains (x / rms * w); "sandwich_vector": the sandwich form with such vector gains;
     # "parallel_dyt": x <- x + residual_mult * (mixer(norm1(x)) + ff(norm2(x))), both sublayers on the same x, every norm (the final
     # one too) a Dynamic Tanh tanh(alpha x) * w + b with the tensors <name>, <name>.alpha, <name>.b; "post": the norm comes after the sum,
     # x <- norm1(post_alpha * x + mixer(x)), then x <- norm2(post_alpha * x + ff(x)), the sublayers read x itself and every norm has a
@@ -261,11 +296,23 @@ class SeqLMConfig:
     # what goes on to the next layer (and to the output) is sum_j dwa[j] X_j over the embedding output X_0 and the results X_1 ..
     # X_(i+1) of the layers so far (the layer's tensor dwa [i + 2])
     depth_average: bool = False
+    # > 0: hyper-connections (pre-norm forms).  Instead of one x there are that many copies x_s, all the embedding output at first; for
+    # sublayer q (1: mixer, 2: feed-forward) u = sum_s hc<q>.in[s] x_s, y = sublayer(norm(u)), then, all from the old copies,
+    # x_t <- sum_s hc<q>.mix[s, t] x_s + hc<q>.out[t] y; the output reads the sum of the copies
+    streams: int = 0
+    learned_positions: int = 0     # > 0: the learned vector pos[p] is added to the (scaled) embedding; a request is at most that long
+    logit_scale: float = 1.0
 
 
 # the weight of every mixer's first product of its operand (SeqLMWeights)
 FIRST_PRODUCT = {RetentionConfig: "w_qkvg", LatentAttentionConfig: "w_qdkv", WindowAttentionConfig: "w_qkv", MinGRUConfig: "w_zxg",
-                 MLSTMConfig: "w_proj"}
+                 MLSTMConfig: "w_proj", GatedLinearConfig: "w_proj"}
+WKV_MIXES = ("r", "k", "v", "g", "w")      # the order of a WKV mixer's operands and projections
+
+
+def _pad_rows(t: torch.Tensor, n: int) -> torch.Tensor:
+    """zero rows up to n (a projection of the same operand as its neighbours whose last columns nobody reads)"""
+    return t if t.shape[0] >= n else torch.cat([t, torch.zeros(n - t.shape[0], t.shape[1], dtype=t.dtype, device=t.device)], 0)
 
 
 def softplus(x: float) -> float:
@@ -300,9 +347,15 @@ class SeqLMWeights:
         def one_plus(layer, key):           # a gain stored around zero
             return (1.0 + w(layer, key, (cfg.width,)).float()).contiguous().to(dev)
 
-        if cfg.norm not in ("sandwich", "pre", "sandwich_vector", "parallel_dyt", "post"):
+        if cfg.norm not in ("sandwich", "pre", "pre_plain", "sandwich_vector", "parallel_dyt", "post"):
             raise ValueError(f"unknown norm style {cfg.norm!r}")
-        pre = cfg.norm == "pre"
+        plain = cfg.norm in ("post", "pre_plain")      # gains stored as they are
+        if cfg.streams and (cfg.norm not in ("pre", "pre_plain") or cfg.residual_mult != 1.0
+                            or any(lc.token_shift or lc.input_conv or lc.add_before is not None for lc in cfg.layers)):
+            raise ValueError("hyper-connections go with the pre-norm layer forms without residual multiplier, token shift, input convolution or added vectors")
+        if any(isinstance(lc.mixer, WKVConfig) and (lc.token_shift or lc.input_conv or cfg.norm in ("parallel_dyt", "post")) for lc in cfg.layers):
+            raise ValueError("a WKV mixer shifts its own input: no token shift, input convolution, parallel or post-norm layers around it")
+        pre = cfg.norm in ("pre", "pre_plain")
         dyt = cfg.norm == "parallel_dyt"
         post = cfg.norm == "post"
         if post and any(lc.token_shift or lc.add_before is not None for lc in cfg.layers):
@@ -319,7 +372,12 @@ class SeqLMWeights:
         D = cfg.width
         self.embed = mat(w(None, "embed", (cfg.vocab, D)))
         self.head = mat(w(None, "head", (cfg.vocab, D)))
-        self.final_gain = dyt_norm(None, "final.norm") if dyt else vec(w(None, "final.norm", (D,))) if post else one_plus(None, "final.norm") if vector else num(None, "final.norm")
+        self.final_gain = dyt_norm(None, "final.norm") if dyt else vec(w(None, "final.norm", (D,))) if plain else one_plus(None, "final.norm") if vector else num(None, "final.norm")
+        if cfg.logit_scale != 1.0:      # the factor of the logits rides on the last norm
+            self.final_gain = ((self.final_gain[0], self.final_gain[1] * cfg.logit_scale, self.final_gain[2] * cfg.logit_scale) if dyt
+                               else self.final_gain * cfg.logit_scale)
+        if cfg.learned_positions:
+            self.pos = mat(w(None, "pos", (cfg.learned_positions, D)))
         if cfg.position_base > 0:      # frequencies in float64, split into two floats hi + lo
             f64 = cfg.position_base ** (-2.0 * np.arange((D + 1) // 2, dtype=np.float64) / D)
             hi = f64.astype(np.float32)
@@ -348,7 +406,7 @@ class SeqLMWeights:
                 continue
             if dyt:
                 lw: Dict[str, object] = {"norm1": dyt_norm(i, "norm1")}
-            elif post:
+            elif plain:
                 lw = {"norm1": vec(w(i, "norm1", (D,)))}
             elif pre:
                 lw = {"norm1": one_plus(i, "norm1")}
@@ -356,14 +414,45 @@ class SeqLMWeights:
                 lw = {k: one_plus(i, k) for k in ("norm1", "norm1b")}
             else:
                 lw = {k: num(i, k) for k in ("norm1", "norm1b")}
+            if cfg.streams:
+                for q in ("hc1", "hc2") if lc.ff is not None else ("hc1",):
+                    lw[q] = (vec(w(i, q + ".in", (cfg.streams,))), vec(w(i, q + ".mix", (cfg.streams, cfg.streams))), vec(w(i, q + ".out", (cfg.streams,))))
             if lc.token_shift:
                 lw["shift"] = vec(w(i, "shift", (D,)))
             if lc.input_conv:      # [taps][width]: the lanes of a kernel read neighbouring channels of one tap
                 for k in ("conv1", "conv2") if lc.ff is not None else ("conv1",):
                     lw[k] = vec(w(i, k, (D, lc.input_conv)).t())
+            def low_rank(mw, first, second, bias):
+                """the two factors of a decay's pre-activation: `second` also written twice side by side for a split operand"""
+                rank, n = first.shape[0], second.shape[0]
+                mw["rank"], mw["w2"], mw["z_bias"] = rank, mat(second), vec(bias.reshape(n))
+                if rank >= 32 and n >= PAD_PROJECTION_ROWS:
+                    mw["w2_split"] = mat(torch.cat([second, second], 1))
+
             def mixer_weights(m, pfx: str) -> Dict[str, object]:
                 """the tensors of one mixer, named <pfx><key> in the checkpoint"""
                 mw: Dict[str, object] = {}
+                if isinstance(m, WKVConfig):
+                    n = m.heads * m.dim
+                    w1 = w(i, pfx + "w1")
+                    low_rank(mw, w1, w(i, pfx + "w2", (n, w1.shape[0])), w(i, pfx + "w0", (n,)))
+                    if n >= PAD_PROJECTION_ROWS:
+                        w1 = _pad_rows(w1, PAD_PROJECTION_ROWS)
+                    # one weight [r | k | v | g | w1] for one product whose column groups read operands of their own
+                    mw["w_proj"] = mat(torch.cat([w(i, pfx + s, (n, D)) for s in "rkvg"] + [w1], 0))
+                    mw["mu"] = vec(torch.stack([w(i, pfx + "mu." + s, (D,)) for s in WKV_MIXES], 0))
+                    mw["bonus"] = vec(w(i, pfx + "u", (m.heads, m.dim)).reshape(n))
+                    mw["out_gain"] = vec(w(i, pfx + "norm", (n,)))
+                    mw["w_o"] = mat(w(i, pfx + "o", (D, n)))
+                    return mw
+                if isinstance(m, GatedLinearConfig):
+                    n, e = m.heads * m.dim, m.heads * m.vdim
+                    a1 = w(i, pfx + "a1")
+                    low_rank(mw, a1, w(i, pfx + "a2", (n, a1.shape[0])), w(i, pfx + "a2.b", (n,)))
+                    mw["w_proj"] = mat(torch.cat([w(i, pfx + "q", (n, D)), w(i, pfx + "k", (n, D)), w(i, pfx + "v", (e, D)), w(i, pfx + "g", (e, D)), a1], 0))
+                    mw["out_gain"] = vec(w(i, pfx + "norm", (m.vdim,)))
+                    mw["w_o"] = mat(w(i, pfx + "o", (D, e)))
+                    return mw
                 if not isinstance(m, (MinGRUConfig, MLSTMConfig)):
                     inv_freq, mag = rotary_table(m.rot)
                     mw["inv_freq"], mw["rot_mag"] = inv_freq.to(dev), mag
@@ -382,8 +471,17 @@ class SeqLMWeights:
                     if m.heads % m.kv_heads:
                         raise ValueError(f"layer {i}: {m.heads} query heads over {m.kv_heads} key / value heads")
                     parts = [w(i, pfx + "q", (m.heads * m.dim, D))]
+                    if m.values_are_keys and (m.vdim != m.dim or m.bias or m.value_norm or m.value_rot is not None):
+                        raise ValueError(f"layer {i}: values that are the keys have the keys' size and no bias, norm or rotation of their own")
+                    if m.qk_conv and m.kv_from is not None:
+                        raise ValueError(f"layer {i}: a convolution over the keys needs keys of the layer's own")
                     if m.kv_from is None:
-                        parts += [w(i, pfx + "k", (m.kv_heads * m.dim, D)), w(i, pfx + "v", (m.kv_heads * m.vdim, D))]
+                        parts.append(w(i, pfx + "k", (m.kv_heads * m.dim, D)))
+                        if not m.values_are_keys:
+                            parts.append(w(i, pfx + "v", (m.kv_heads * m.vdim, D)))
+                    if m.qk_conv:      # [taps][q channels | k channels]
+                        mw["qk_conv"] = vec(torch.cat([w(i, pfx + "q.conv", (m.heads * m.dim, m.qk_conv)),
+                                                       w(i, pfx + "k.conv", (m.kv_heads * m.dim, m.qk_conv))], 0).t())
                     if m.out_gate:
                         parts.append(w(i, pfx + "g", (m.heads * m.vdim, D)))
                     mw["w_qkv"] = mat(torch.cat(parts, 0))
@@ -395,16 +493,18 @@ class SeqLMWeights:
                         mw["o_bias"] = vec(w(i, pfx + "o.b", (D,)))
                     if m.talking_heads:
                         mw["talk"] = vec(w(i, pfx + "talk", (m.heads, m.heads)))
-                    elif m.out_gate:      # the gate rides on the mixing kernel: no mixing is the unit matrix
-                        mw["talk"] = torch.eye(m.heads, dtype=F32).to(dev)
                     if m.head_temp:
                         mw["temp"] = vec(w(i, pfx + "temp", (m.heads,)))
                     if m.distance_bias:
-                        if m.pool or m.talking_heads or m.out_gate:
-                            raise ValueError(f"layer {i}: a distance bias with pooled blocks or with mixed or gated heads is not supported")
+                        if m.pool or m.talking_heads or m.distance_slope:
+                            raise ValueError(f"layer {i}: a distance bias with pooled blocks, mixed heads or a second bias is not supported")
                         mw["dist_amp"], mw["dist_rate"] = vec(w(i, pfx + "r1", (m.heads,))), vec(w(i, pfx + "r2", (m.heads,)))
-                    if (m.talking_heads or m.out_gate) and m.value_rot is not None:
-                        raise ValueError(f"layer {i}: mixed or gated heads with rotated values are not supported")
+                    if m.distance_slope:
+                        if m.pool or m.talking_heads:
+                            raise ValueError(f"layer {i}: a distance bias with pooled blocks or mixed heads is not supported")
+                        mw["dist_amp"] = torch.tensor([2.0 ** (-8.0 * (hd + 1) / m.heads) for hd in range(m.heads)], dtype=torch.float64).to(F32).to(dev)
+                    if m.talking_heads and m.value_rot is not None:
+                        raise ValueError(f"layer {i}: mixed heads with rotated values are not supported")
                     if m.qk_norm == "head":      # a layer without keys of its own hands the kernel its query gain twice (the second is unused)
                         mw["q_gain"] = vec(w(i, pfx + "q.norm", (m.dim,)))
                         mw["k_gain"] = vec(w(i, pfx + "k.norm", (m.dim,))) if m.kv_from is None else mw["q_gain"]
@@ -458,9 +558,28 @@ class SeqLMWeights:
                     if isinstance(sub, ParallelMixerConfig) or getattr(sub, "kv_from", None) is not None:
                         raise ValueError(f"layer {i}: a branch of a parallel mixer is a plain mixer with a cache of its own")
                     lw[side] = mixer_weights(sub, f"mix.{side}.")
+                    if isinstance(sub, WKVConfig):
+                        raise ValueError(f"layer {i}: a WKV mixer is not a branch of a parallel one")
+                    if m.scales is not None:
+                        continue
                     lw[side + "_out"] = (0.5 * w(i, f"mix.{side}.out", (D,)).float()).contiguous().to(dev)      # the halving rides on the gain
+                if m.scales is not None:
+                    if not isinstance(m.left, WindowAttentionConfig) or not isinstance(m.right, GatedLinearConfig) or m.left.talking_heads or m.left.out_bias:
+                        raise ValueError(f"layer {i}: a scaled parallel mixer is window attention beside gated linear attention")
+                    # one product for both branches' projections and one for both outputs (left's scale rides on its kernel's store,
+                    # right's on its gain)
+                    first = torch.cat([lw["left"]["w_qkv"], lw["right"]["w_proj"]], 0)
+                    lw["w_in"] = _pad_rows(first, -(-first.shape[0] // 8) * 8 if first.shape[0] >= PAD_PROJECTION_ROWS else 0).contiguous()
+                    n_left = lw["left"]["w_qkv"].shape[0]
+                    lw["in_split"] = [(0, n_left), (n_left, first.shape[0] - n_left)]
+                    lw["w_o"] = torch.cat([lw["left"]["w_o"], lw["right"]["w_o"]], 1).contiguous()
+                    lw["right"]["out_gain"] = lw["right"]["out_gain"] * m.scales[1]
+                    for side, key in (("left", "w_qkv"), ("right", "w_proj")):
+                        del lw[side][key], lw[side]["w_o"]
             else:
                 lw.update(mixer_weights(m, "mix."))
+            if cfg.residual_gate and isinstance(m, ParallelMixerConfig) and m.scales is not None:
+                raise ValueError(f"layer {i}: gated branches around a scaled parallel mixer are not supported")
             if cfg.residual_gate:
                 lw["w_rg1"], lw["rg1_bias"] = mat(w(i, "rg1", (D, D))), vec(w(i, "rg1.b", (D,)))
                 # the mixer's first projections and its gate read the same operand: one weight [projections | gate] and one product;
@@ -483,7 +602,7 @@ class SeqLMWeights:
                 lw["dwa"] = vec(w(i, "dwa", (i + 2,)))
             f = lc.ff
             if f is not None:
-                lw.update({"norm2": dyt_norm(i, "norm2")} if dyt else {"norm2": vec(w(i, "norm2", (D,)))} if post else {"norm2": one_plus(i, "norm2")} if pre else
+                lw.update({"norm2": dyt_norm(i, "norm2")} if dyt else {"norm2": vec(w(i, "norm2", (D,)))} if plain else {"norm2": one_plus(i, "norm2")} if pre else
                           {k: (one_plus(i, k) if vector else num(i, k)) for k in ("norm2", "norm2b")})
             if isinstance(f, DenseFFConfig) and f.act in ("clamp_glu", "gelu_glu"):
                 lw["w_gu"] = mat(torch.cat([w(i, "mlp.gate", (f.ff, D)), w(i, "mlp.up", (f.ff, D))], 0))
@@ -507,6 +626,9 @@ class SeqLMWeights:
                 elif f.router == "sigmoid_input":
                     if f.n_groups != 1:
                         raise ValueError(f"layer {i}: the plain sigmoid router has no groups")
+                elif f.router == "group_softmax":
+                    if f.shared_ff and f.shared_gate:
+                        raise ValueError(f"layer {i}: the group softmax router has no gate for a shared expert")
                 elif f.router != "grouped_sigmoid":
                     raise ValueError(f"layer {i}: unknown router {f.router!r}")
                 else:
@@ -644,6 +766,9 @@ class SeqLMEngine:
         # The tables are keyed by the layer, or by (layer, "left" | "right") for the branches of a parallel mixer.
         rows, states, summaries, looks, keep = [], [], [], [], 0
         self._cache_index, self._state_index, self._summary_index, self._shift_index, self._conv_index = {}, {}, {}, [], {}
+        self._prev_index = {}          # the previous token's input of a WKV mixer
+        if cfg.streams > int(self.L.lp_hyper_max_streams()):
+            raise ValueError(f"{cfg.streams} streams are not built")
 
         def look_back(m):      # how far back a windowed or block-local layer reads (None: everything)
             bounds = [v for v in (m.window, getattr(m, "chunk", None)) if v and v > 0]
@@ -657,7 +782,7 @@ class SeqLMEngine:
                 src = cfg.layers[j].mixer if 0 <= j < len(cfg.layers) and not isinstance(key, tuple) and j < key else None
                 if type(src) is not type(m) or src.kv_from is not None:
                     raise ValueError(f"layer {key}: kv_from = {j} must name an earlier attention layer of its kind that has keys and values of its own")
-                same = ("kv_rank", "rot_dim", "rot") if isinstance(m, LatentAttentionConfig) else ("kv_heads", "dim", "vdim", "rot")
+                same = ("kv_rank", "rot_dim", "rot") if isinstance(m, LatentAttentionConfig) else ("kv_heads", "dim", "vdim", "rot", "values_are_keys")
                 if any(getattr(src, k) != getattr(m, k) for k in same) or (
                         isinstance(m, WindowAttentionConfig) and (m.pool or src.value_rot or m.value_rot)):
                     raise ValueError(f"layer {key}: its key / value sizes and rotation differ from those of layer {j}, whose cache it reads")
@@ -670,11 +795,16 @@ class SeqLMEngine:
                 looks.append(look_back(m))
             elif isinstance(m, WindowAttentionConfig):
                 ci = len(rows)
-                rows.append(m.kv_heads * (m.dim + m.vdim))
+                rows.append(m.kv_heads * (m.dim + (0 if m.values_are_keys else m.vdim)))
+                if m.qk_conv > int(self.L.lp_causal_conv_max_taps()):
+                    raise ValueError(f"layer {key}: a convolution of {m.qk_conv} taps is not built")
+                if m.qk_conv > 1:      # the last taps - 1 projected queries and keys
+                    self._conv_index[(key, "qk")] = len(states)
+                    states.append((m.qk_conv - 1, (m.heads + m.kv_heads) * m.dim))
                 windowed = bool(m.window and m.window > 0)
                 if windowed and m.pool > 0:
                     pi = len(summaries)
-                    summaries.append((m.kv_heads * (m.dim + m.vdim), m.pool))
+                    summaries.append((rows[ci], m.pool))
                 # a pooled layer reads a block's tokens once more when the block is complete
                 looks.append(max(m.window, m.pool) if windowed and m.pool > 0 else look_back(m))
                 keep = max(keep, m.keep_first if windowed else 0)
@@ -687,6 +817,12 @@ class SeqLMEngine:
             elif isinstance(m, MLSTMConfig):
                 si = len(states)
                 states.append((m.heads, m.dim + 1, m.vdim + 1))      # per head S | n, and the running maximum in the last row
+            elif isinstance(m, (WKVConfig, GatedLinearConfig)):
+                si = len(states)
+                states.append((m.heads, m.dim, m.dim if isinstance(m, WKVConfig) else m.vdim))
+                if isinstance(m, WKVConfig):
+                    self._prev_index[key] = len(states)
+                    states.append((cfg.width,))
             else:
                 raise TypeError(f"unknown mixer {type(m).__name__}")
             self._cache_index[key], self._state_index[key], self._summary_index[key] = ci, si, pi
@@ -782,6 +918,24 @@ class SeqLMEngine:
         self._check(self.L.lp_linear(C.byref(d), self._stream()), "lp_linear")
         return out
 
+    def linear_segments(self, ops: torch.Tensor, w: torch.Tensor, seg: int) -> torch.Tensor:
+        """fp32 [R, N]: columns [i seg, (i + 1) seg) are ops[i] @ w[those rows].T, the last operand takes all that follow (ops [S, R, D])"""
+        S, R, D = ops.shape
+        N = w.shape[0]
+        bounds = [i * seg for i in range(S)] + [N]
+        out = self._empty((R, N), F32)
+        parts = [(ops[i], w[a:b], out[:, a:b]) for i, (a, b) in enumerate(zip(bounds, bounds[1:]))]
+        fits = seg % (_lib.LINEAR_ROWS_COLS if R <= _lib.LINEAR_ROWS_MAX else self.tile_rows) == 0
+        if not fits or any(self._on_tensor_cores(a, wi, R, wi.shape[0], D) for a, wi, _ in parts):
+            for a, wi, o in parts:
+                self.linear(a, wi, F32, out=o)
+            return out
+        d = _lib.LinearDesc(A=_lib.ptr(ops), lda=ops.stride(1), a_batch=0, a_fp32=int(ops.dtype == F32), W=_lib.ptr(w), ldw=w.stride(0),
+                            w_batch=0, C=_lib.ptr(out), ldc=N, c_batch=0, c_fp32=1, M=R, N=N, K=D, batch=1, epi=_lib.EPI_NONE,
+                            seg_cols=seg, n_segs=S, a_seg=ops.stride(0))
+        self._check(self.L.lp_linear(C.byref(d), self._stream()), "lp_linear")
+        return out
+
     def linear_heads(self, a: torch.Tensor, a_head: int, w: torch.Tensor, out: torch.Tensor, out_head: int, gate=None):
         """Per head h: out[:, h*out_head : +N] = a[:, h*a_head : +K] @ w[h].T with w [heads, N, K]; gate (fp32 rows, N per head): the
         result is multiplied by its sigmoid."""
@@ -821,13 +975,15 @@ class SeqLMEngine:
         """h + conv(h) in the operand dtype for the sublayer `which` of layer li (h: fp32 rows); its carried inputs move on"""
         taps, w = self.cfg.layers[li].input_conv, self.w.layers[li][which]
         out = self._empty(h.shape, self.act)
-        state = self._conv_state(li, which)
-        rc = self.L.lp_causal_conv_f32(_lib.ptr(h), h.stride(0), _lib.ptr(w), taps, h.shape[1], b.n_chunks, _lib.ptr(b.chunk_seq),
+        self._conv(h, w, taps, True, self._conv_state(li, which), out, b)
+        return out
+
+    def _conv(self, h, w, taps, add_input, state, out, b: _Batch) -> None:
+        rc = self.L.lp_causal_conv_f32(_lib.ptr(h), h.stride(0), _lib.ptr(w), taps, int(add_input), h.shape[1], b.n_chunks, _lib.ptr(b.chunk_seq),
                                        _lib.ptr(b.chunk_row0), _lib.ptr(b.chunk_len), b.longest_chunk, _lib.ptr(b.row_pos),
                                        _lib.ptr(b.seq_row0), _lib.ptr(b.seq_slot), _lib.ptr(state), state.stride(0) if state is not None else 0,
                                        _lib.ptr(out), out.stride(0), int(out.dtype == F32), self._stream())
         self._check(rc, "lp_causal_conv_f32")
-        return out
 
     def _conv_state(self, li: int, which: str) -> Optional[torch.Tensor]:
         j = self._conv_index.get((li, which))
@@ -837,7 +993,8 @@ class SeqLMEngine:
         """what a sublayer of a layer with norms ahead of it reads: the normed stream, convolved when the layer says so"""
         if self.cfg.layers[li].input_conv:
             return self.convolved(self.norm(x, gain, F32), li, which, b)
-        return self.norm(x, gain, self.act)
+        wkv = which == "conv1" and isinstance(self.cfg.layers[li].mixer, WKVConfig)      # it shifts its input, in fp32
+        return self.norm(x, gain, F32 if wkv else self.act)
 
     # ------------------------------------------------------------------ mixers
     def _retention(self, li, m: RetentionConfig, lw, h: torch.Tensor, b: _Batch, into=None, proj=None) -> torch.Tensor:
@@ -908,8 +1065,28 @@ class SeqLMEngine:
         return self.linear(o, lw["w_o"], F32, into=into)
 
     def _window_attention(self, li, m: WindowAttentionConfig, lw, h: torch.Tensor, b: _Batch, into=None, proj=None) -> torch.Tensor:
+        o = self._empty((b.R, m.heads * m.vdim), self.act)
+        self._window_heads(li, m, lw, h, b, o, proj)
+        return self.linear(o, lw["w_o"], F32, into=into, bias=lw.get("o_bias"))
+
+    def _window_heads(self, li, m: WindowAttentionConfig, lw, h, b: _Batch, o: torch.Tensor, proj=None, out_scale: float = 1.0) -> None:
+        """the concatenated heads (gated, times out_scale) into o, possibly columns of a wider buffer"""
         qkv = proj if proj is not None else self.linear(h, lw["w_qkv"], F32)      # a layer that reads another layer's keys and values projects its queries only
         hq, hk = m.heads * m.dim, m.kv_heads * m.dim if m.kv_from is None else 0
+        hv = m.kv_heads * m.vdim if m.kv_from is None and not m.values_are_keys else 0
+        gate = qkv[:, hq + hk + hv:] if m.out_gate and not m.talking_heads else None
+        conv = {}
+        if m.qk_conv:
+            state = self._conv_state(li, "qk")
+            if b.decode:      # rides on the preparation of the one row
+                conv = dict(conv_w=_lib.ptr(lw["qk_conv"]), conv_taps=m.qk_conv, row_slot=_lib.ptr(b.seq_slot), conv_state=_lib.ptr(state),
+                            conv_stride=state.stride(0) if state is not None else 0)
+            else:
+                raw = qkv
+                qkv = self._empty((b.R, hq + hk + hv), F32)
+                self._conv(raw[:, :hq + hk], lw["qk_conv"], m.qk_conv, False, state, qkv[:, :hq + hk], b)
+                if hv:
+                    qkv[:, hq + hk:].copy_(raw[:, hq + hk:hq + hk + hv])
         cache = self.cache
         pool = cache.pools[self._cache_index[li]]
         windowed = bool(m.window and m.window > 0)
@@ -917,14 +1094,14 @@ class SeqLMEngine:
         stream = cache.summary_index[pi][0] if pi >= 0 else -1
         layouts = {"half": _lib.ROT_HALF, "interleaved": _lib.ROT_INTERLEAVED}
         vr = m.value_rot
-        mixing = m.talking_heads or m.out_gate
+        mixing = m.talking_heads
         d = _lib.WindowAttnDesc(
             qkv=_lib.ptr(qkv), ld=qkv.stride(0), q_off=0, k_off=hq, v_off=hq + hk, heads=m.heads, kv_heads=m.kv_heads, dim=m.dim,
             vdim=m.vdim,
             norm_mode={"none": _lib.QKNORM_NONE, "head": _lib.QKNORM_HEAD, "unit": _lib.QKNORM_HEAD, "full": _lib.QKNORM_FULL}[m.qk_norm],
             q_bias=_lib.ptr(lw.get("q_bias")), k_bias=_lib.ptr(lw.get("k_bias")), v_bias=_lib.ptr(lw.get("v_bias")),
             v_norm=int(m.value_norm), talk=_lib.ptr(lw.get("talk")),
-            g_off=hq + hk + (m.kv_heads * m.vdim if m.kv_from is None else 0) if m.out_gate else -1,
+            g_off=hq + hk + hv if m.out_gate and mixing else -1,
             q_gain=_lib.ptr(lw.get("q_gain")), k_gain=_lib.ptr(lw.get("k_gain")), eps=self.cfg.eps, inv_freq=_lib.ptr(lw["inv_freq"]),
             rot_dims=m.rot.dims, rot_layout=layouts[m.rot.layout], rot_mscale=lw["rot_mag"],
             v_inv_freq=_lib.ptr(lw.get("v_inv_freq")), v_rot_dims=vr.dims if vr else 0, v_rot_layout=layouts[vr.layout] if vr else 0,
@@ -934,7 +1111,9 @@ class SeqLMEngine:
             max_pooled_pages=b.summary_width[stream] if pi >= 0 else 0, pool=m.pool if pi >= 0 else 0,
             window=m.window if windowed else 0, keep_first=m.keep_first if windowed else 0, scale=m.scale, softcap=m.softcap,
             sink=int(m.sink), chunk=m.chunk or 0, kv_shared=int(m.kv_from is not None), q_temp=_lib.ptr(lw.get("temp")),
-            dist_amp=_lib.ptr(lw.get("dist_amp")), dist_rate=_lib.ptr(lw.get("dist_rate")))
+            dist_amp=_lib.ptr(lw.get("dist_amp")), dist_rate=_lib.ptr(lw.get("dist_rate")), v_is_k=int(m.values_are_keys),
+            gate=_lib.ptr(gate), ldg=gate.stride(0) if gate is not None else 0, out_scale=out_scale,
+            pos_temp_coef=m.pos_temp[0] if m.pos_temp else 0.0, pos_temp_every=m.pos_temp[1] if m.pos_temp else 0, **conv)
         st = self._stream()
         self._check(self.L.lp_window_attn_prep(C.byref(d), b.R, _lib.ptr(b.row_seq), _lib.ptr(b.row_pos), st), "lp_window_attn_prep")
         if pi >= 0:
@@ -942,7 +1121,6 @@ class SeqLMEngine:
             new = 1 if b.decode else b.summary_new[stream]
             rc = self.L.lp_window_attn_pool(C.byref(d), b.n, _lib.ptr(b.seq_row0), _lib.ptr(b.seq_pos0), new, st)
             self._check(rc, "lp_window_attn_pool")
-        o = self._empty((b.R, m.heads * m.vdim), self.act)
         if mixing and b.decode:      # weights mixed over the heads (and the output gate): a CTA per row
             rc = self.L.lp_window_attn_talk(C.byref(d), b.R, _lib.ptr(b.row_seq), _lib.ptr(b.row_pos), _lib.ptr(o), o.stride(0),
                                             int(o.dtype == F32), st)
@@ -957,7 +1135,68 @@ class SeqLMEngine:
             rc = self.L.lp_window_attn_tiles(C.byref(d), b.R, _lib.ptr(b.row_seq), _lib.ptr(b.row_pos), b.n_chunks, _lib.ptr(b.chunk_seq),
                                              _lib.ptr(b.chunk_row0), _lib.ptr(b.chunk_len), _lib.ptr(o), o.stride(0), int(o.dtype == F32), st)
         self._check(rc, "lp_window_attn")
-        return self.linear(o, lw["w_o"], F32, into=into, bias=lw.get("o_bias"))
+
+    def _decay_rows(self, lw, t: torch.Tensor, tanh: bool) -> torch.Tensor:
+        """the pre-activations of a decay, fp32 [R, heads * dim], from its low-rank vector t: a product that keeps its operand's 32 bits — as
+        fp32, or on the tensor cores with the operand split into two bf16 halves"""
+        R, rank, st = t.shape[0], lw["rank"], self._stream()
+        w2 = lw.get("w2_split")
+        split = w2 is not None and self.tensor_core_rows is not None and R >= self.tensor_core_rows and rank % 4 == 0 and w2.shape[0] % 8 == 0
+        if split or tanh:
+            a = self._empty((R, 2 * rank), BF16) if split else self._empty((R, rank), F32)
+            rc = self.L.lp_lowrank_operand(_lib.ptr(t), t.stride(0), R, rank, int(tanh), _lib.ptr(a), a.stride(0), int(split), st)
+            self._check(rc, "lp_lowrank_operand")
+            t = a
+        return self.linear(t, w2 if split else lw["w2"], F32, bias=lw["z_bias"])
+
+    def _decayed_memory(self, li, lw, b: _Batch, out: torch.Tensor, heads: int, dim: int, vdim: int, q, k, v, gate, t, tanh: bool, **form) -> None:
+        """the matrix memory with a decay per key channel: q, k, v, gate and the decay's low-rank vector t are column ranges of fp32 rows"""
+        state = self.cache.states[self._state_index[li]]
+        d = _lib.GlaDesc(q=_lib.ptr(q), k=_lib.ptr(k), v=_lib.ptr(v), ldq=q.stride(0), ldk=k.stride(0), ldv=v.stride(0), heads=heads, dim=dim,
+                         vdim=vdim, gate=_lib.ptr(gate), ldg=gate.stride(0), eps=self.cfg.eps, out_gain=_lib.ptr(lw["out_gain"]),
+                         state=_lib.ptr(state), slot_stride=state.stride(0), out=_lib.ptr(out), ldo=out.stride(0), out_fp32=int(out.dtype == F32), **form)
+        if b.decode:      # the decays of one row are made where they are used
+            d.t, d.ldt, d.w2, d.ldw2, d.rank, d.t_tanh, d.z_bias = (_lib.ptr(t), t.stride(0), _lib.ptr(lw["w2"]), lw["w2"].stride(0), lw["rank"],
+                                                                     int(tanh), _lib.ptr(lw["z_bias"]))
+        else:
+            z = self._decay_rows(lw, t, tanh)
+            d.z, d.ldz = _lib.ptr(z), z.stride(0)
+        longest = max(b.lens)
+        nbytes = int(self.L.lp_gla_workspace_bytes(b.n_chunks, b.R, longest, heads, dim, vdim))
+        ws = self._empty((nbytes // 4,), F32) if nbytes else None
+        rc = self.L.lp_gla(C.byref(d), b.n, b.n_chunks, b.R, longest, _lib.ptr(b.seq_row0), _lib.ptr(b.seq_pos0), _lib.ptr(b.seq_slot),
+                           _lib.ptr(b.seq_chunk0), _lib.ptr(b.chunk_seq), _lib.ptr(b.chunk_row0), _lib.ptr(b.chunk_len), _lib.ptr(ws), nbytes,
+                           self._stream())
+        self._check(rc, "lp_gla")
+
+    def _wkv(self, li, m: WKVConfig, lw, h: torch.Tensor, b: _Batch, into=None) -> torch.Tensor:
+        """h: the five mixes [5, R, D] in the operand dtype, or the normed rows [R, D] in fp32, which are shifted and mixed here"""
+        n = m.heads * m.dim
+        if h.dim() == 2:
+            ops = self._empty((len(WKV_MIXES), *h.shape), self.act)
+            state = self.cache.states[self._prev_index[li]]
+            rc = self.L.lp_token_shift_mix_f32(_lib.ptr(h), h.stride(0), _lib.ptr(lw["mu"]), len(WKV_MIXES), b.R, h.shape[1], _lib.ptr(b.row_seq),
+                                               _lib.ptr(b.row_pos), _lib.ptr(b.seq_row0), _lib.ptr(b.seq_slot), _lib.ptr(state), state.stride(0),
+                                               _lib.ptr(ops), ops.stride(1), ops.stride(0), int(ops.dtype == F32), self._stream())
+            self._check(rc, "lp_token_shift_mix_f32")
+            h = ops
+        p = self.linear_segments(h, lw["w_proj"], n)
+        out = self._empty((b.R, n), self.act)
+        self._decayed_memory(li, lw, b, out, m.heads, m.dim, m.dim, p[:, :n], p[:, n:2 * n], p[:, 2 * n:3 * n], p[:, 3 * n:4 * n],
+                             p[:, 4 * n:4 * n + lw["rank"]], True, q_scale=1.0, decay=_lib.GLA_DECAY_DOUBLE_EXP, bonus=_lib.ptr(lw["bonus"]),
+                             gain_stride=m.dim)
+        return self.linear(out, lw["w_o"], F32, into=into)
+
+    def _gated_linear(self, li, m: GatedLinearConfig, lw, h: torch.Tensor, b: _Batch, into=None, proj=None) -> torch.Tensor:
+        out = self._empty((b.R, m.heads * m.vdim), self.act)
+        self._gated_linear_heads(li, m, lw, proj if proj is not None else self.linear(h, lw["w_proj"], F32), b, out)
+        return self.linear(out, lw["w_o"], F32, into=into)
+
+    def _gated_linear_heads(self, li, m: GatedLinearConfig, lw, p: torch.Tensor, b: _Batch, out: torch.Tensor) -> None:
+        n, e = m.heads * m.dim, m.heads * m.vdim
+        self._decayed_memory(li, lw, b, out, m.heads, m.dim, m.vdim, p[:, :n], p[:, n:2 * n], p[:, 2 * n:2 * n + e], p[:, 2 * n + e:2 * n + 2 * e],
+                             p[:, 2 * n + 2 * e:2 * n + 2 * e + lw["rank"]], False, q_scale=m.dim ** -0.5, decay=_lib.GLA_DECAY_SIGMOID_POW,
+                             decay_exp=1.0 / m.tau, gain_stride=0)
 
     def _mingru(self, li, m: MinGRUConfig, lw, h: torch.Tensor, b: _Batch, into=None, proj=None) -> torch.Tensor:
         zxg = proj if proj is not None else self.linear(h, lw["w_zxg"], F32)
@@ -997,7 +1236,16 @@ class SeqLMEngine:
 
     def _parallel(self, li: int, m: ParallelMixerConfig, lw, h: torch.Tensor, b: _Batch, into=None, proj=None) -> torch.Tensor:
         """two mixers on the same input; each output is RMS-normed over the width with its own gain (which carries the halving);
-        proj: the two branches' first products when one product of the layer made them"""
+        proj: the two branches' first products when one product of the layer made them.  With scales: the branches' heads side by side in
+        one buffer, one product for the scaled sum of both"""
+        if m.scales is not None:
+            wide = self.linear(h, lw["w_in"], F32)
+            pl, pr = (wide[:, a:a + n] for a, n in lw["in_split"])
+            nl = m.left.heads * m.left.vdim
+            o = self._empty((b.R, lw["w_o"].shape[1]), self.act)
+            self._window_heads((li, "left"), m.left, lw["left"], None, b, o[:, :nl], pl, out_scale=m.scales[0])
+            self._gated_linear_heads((li, "right"), m.right, lw["right"], pr, b, o[:, nl:])
+            return self.linear(o, lw["w_o"], F32, into=into)
         left = self._mix((li, "left"), m.left, lw["left"], h, b, proj=proj[0] if proj is not None else None)
         right = self._mix((li, "right"), m.right, lw["right"], h, b, proj=proj[1] if proj is not None else None)
         mix = self.norm(left, lw["left_out"], F32)
@@ -1016,6 +1264,10 @@ class SeqLMEngine:
         mixer's first product of h (fp32, possibly columns of a wider product) when the caller has made it already"""
         if isinstance(m, ParallelMixerConfig):
             return self._parallel(li, m, lw, h, b, into, proj)
+        if isinstance(m, WKVConfig):
+            return self._wkv(li, m, lw, h, b, into)
+        if isinstance(m, GatedLinearConfig):
+            return self._gated_linear(li, m, lw, h, b, into, proj)
         if isinstance(m, MLSTMConfig):
             return self._mlstm(li, m, lw, h, b, into, proj)
         if isinstance(m, RetentionConfig):
@@ -1053,6 +1305,10 @@ class SeqLMEngine:
             rc = L.lp_moe_route_softmax(_lib.ptr(h), h.stride(0), int(h.dtype == F32), T, D, _lib.ptr(lw["w_router"]),
                                         lw["w_router"].stride(0), f.experts, _lib.ptr(lw["router_bias"]), f.top, _lib.ptr(idx),
                                         _lib.ptr(wts), st)
+        elif f.router == "group_softmax":
+            rc = L.lp_moe_route_group_softmax(_lib.ptr(h), h.stride(0), int(h.dtype == F32), T, D, _lib.ptr(lw["w_router"]),
+                                              lw["w_router"].stride(0), f.experts, f.n_groups, f.keep_groups, f.top, float(f.weight_scale),
+                                              _lib.ptr(idx), _lib.ptr(wts), st)
         else:
             rc = L.lp_moe_route(_lib.ptr(h), h.stride(0), int(h.dtype == F32), T, D, _lib.ptr(lw["w_router"]), lw["w_router"].stride(0),
                                 f.experts, _lib.ptr(lw["correction"]), f.n_groups, f.keep_groups, f.top,
@@ -1147,6 +1403,11 @@ class SeqLMEngine:
             return None
         if len({e.key for e in entries}) != len(entries):
             raise ValueError("a request appears twice in one step")
+        if self.cfg.learned_positions:
+            for e in entries:
+                s = self.cache.get(e.key)
+                if (s.length if s is not None else 0) + len(e.tokens) > self.cfg.learned_positions:
+                    raise ValueError(f"request {e.key!r} would be longer than the model's {self.cfg.learned_positions} positions")
         b = _Batch(self, entries, self._static_tables if self.use_graphs else None)
         if b.decode and self.use_graphs and self.tap is None:
             logits = self._decode_replay(b)
@@ -1186,6 +1447,17 @@ class SeqLMEngine:
         hist = None
         if cfg.depth_average:      # every layer's result is kept: the embedding output is the first of them
             hist = self._empty((len(cfg.layers) + 1, b.R, D), F32)
+        if cfg.streams or cfg.learned_positions:      # learned positions, and every copy of the stream
+            copies = max(cfg.streams, 1)
+            x = hist[0] if hist is not None else self._empty((b.R, copies * D), F32)
+            pos = self.w.pos if cfg.learned_positions else None
+            rc = self.L.lp_embed_streams_f32(_lib.ptr(b.tokens), b.R, _lib.ptr(self.w.embed), self.w.embed.stride(0), cfg.vocab, cfg.embed_scale,
+                                             _lib.ptr(pos), pos.stride(0) if pos is not None else 0, cfg.learned_positions, _lib.ptr(b.row_pos),
+                                             _lib.ptr(x), x.stride(0), D, copies, self._stream())
+            self._check(rc, "lp_embed_streams_f32")
+            if cfg.streams:
+                return self._forward_streams(b, want, x)
+            return self._layers(b, want, x, hist)
         x = hist[0] if hist is not None else self._empty((b.R, D), F32)
         rc = self.L.lp_embed_rows_f32(_lib.ptr(b.tokens), b.R, _lib.ptr(self.w.embed), self.w.embed.stride(0), cfg.vocab, cfg.embed_scale,
                                       _lib.ptr(x), x.stride(0), D, self._stream())
@@ -1194,11 +1466,16 @@ class SeqLMEngine:
             rc = self.L.lp_add_positions_f32(_lib.ptr(x), x.stride(0), b.R, D, _lib.ptr(b.row_pos), _lib.ptr(self.w.position_freq),
                                              self._stream())
             self._check(rc, "lp_add_positions_f32")
+        return self._layers(b, want, x, hist)
+
+    def _layers(self, b: _Batch, want, x: torch.Tensor, hist) -> Optional[torch.Tensor]:
+        """the layers of a model with one stream, in the form of its norms"""
+        cfg, D = self.cfg, self.cfg.width
         if cfg.norm == "parallel_dyt":
             return self._forward_parallel(b, want, x, hist)
         if cfg.norm == "post":
             return self._forward_post(b, want, x)
-        pre = cfg.norm == "pre"
+        pre = cfg.norm in ("pre", "pre_plain")
         for li, (lc, lw) in enumerate(zip(cfg.layers, self.w.layers)):
             if self.w.add_before[li] is not None:
                 rc = self.L.lp_add_row_f32(_lib.ptr(x), x.stride(0), _lib.ptr(self.w.add_before[li]), b.R, D, self._stream())
@@ -1240,6 +1517,47 @@ class SeqLMEngine:
         rows = x if isinstance(want, str) else x.index_select(0, want.long())
         hn = self.dyt(rows, self.w.final_gain)[0] if self.cfg.norm == "parallel_dyt" else self.norm(rows, self.w.final_gain, self.act)
         return self.linear(hn, self.w.head, F32)
+
+    def _hyper(self, x: torch.Tensor, b: _Batch, closes=None, opens=None, wkv=None) -> Optional[torch.Tensor]:
+        """x [R, streams * D] in place.  closes: (y, mix, out weights) of the sublayer that has run; opens: (in weights or None, gain) of the
+        next one, whose operand is returned.  wkv: key of a WKV mixer that reads it — its mixes in one-token steps, else the fp32 rows"""
+        cfg, R, D = self.cfg, b.R, self.cfg.width
+        d = _lib.HyperDesc(x=_lib.ptr(x), ldx=x.stride(0), n=cfg.streams, D=D, eps=cfg.eps)
+        if closes is not None:
+            y, mix, out_w = closes
+            d.y, d.ldy, d.mix, d.out_w = _lib.ptr(y), y.stride(0), _lib.ptr(mix), _lib.ptr(out_w)
+        h = None
+        if opens is not None:
+            d.in_w, d.gain = _lib.ptr(opens[0]), _lib.ptr(opens[1])
+            if wkv is not None and b.decode:
+                mu, state = self.w.layers[wkv]["mu"], self.cache.states[self._prev_index[wkv]]
+                h = self._empty((mu.shape[0], R, D), self.act)
+                d.mu, d.n_mix, d.mix_stride, d.row_pos, d.row_slot = _lib.ptr(mu), mu.shape[0], h.stride(0), _lib.ptr(b.row_pos), _lib.ptr(b.seq_slot)
+                d.state, d.slot_stride = _lib.ptr(state), state.stride(0)
+            else:
+                h = self._empty((R, D), F32 if wkv is not None else self.act)
+            d.h, d.ldh, d.h_fp32 = _lib.ptr(h), D, int(h.dtype == F32)
+        self._check(self.L.lp_hyper_f32(C.byref(d), R, self._stream()), "lp_hyper_f32")
+        return h
+
+    def _forward_streams(self, b: _Batch, want, x: torch.Tensor) -> Optional[torch.Tensor]:
+        """Hyper-connected layers: one kernel between two sublayers closes the one and opens the other in one pass over the copies."""
+        cfg = self.cfg
+        pending = None
+        for li, (lc, lw) in enumerate(zip(cfg.layers, self.w.layers)):
+            h = self._hyper(x, b, pending, (lw["hc1"][0], lw["norm1"]), wkv=li if isinstance(lc.mixer, WKVConfig) else None)
+            pending = (self._mix(li, lc.mixer, lw, h, b), *lw["hc1"][1:])
+            if lc.ff is not None:
+                h = self._hyper(x, b, pending, (lw["hc2"][0], lw["norm2"]))
+                pending = (self._dense(lc.ff, lw, h) if isinstance(lc.ff, DenseFFConfig) else self._moe(lc.ff, lw, h), *lw["hc2"][1:])
+            if self.tap is not None:
+                self._hyper(x, b, pending)
+                pending = None
+                self.tap(li, x.view(b.R, cfg.streams, cfg.width).sum(1))
+        if want is None:
+            return None
+        h = self._hyper(x, b, pending, (None, self.w.final_gain))      # the sum of the copies, normed
+        return self.linear(h if isinstance(want, str) else h.index_select(0, want.long()), self.w.head, F32)
 
     def _forward_post(self, b: _Batch, want, x: torch.Tensor) -> Optional[torch.Tensor]:
         """Layers whose norm follows the sum: x <- norm(post_alpha x + sublayer(x)).  One kernel closes a sublayer and writes the operand

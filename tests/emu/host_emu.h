@@ -85,6 +85,8 @@ inline void note_launch(int = 1) {}
 inline void pdl_wait() {}
 inline void pdl_launch_dependents() {}
 inline int sm_count() { return 4; }
+inline float2 fma2(float2 a, float2 b, float2 c) { return {std::fma(a.x, b.x, c.x), std::fma(a.y, b.y, c.y)}; }
+inline float2 mul2(float2 a, float2 b) { return {a.x * b.x, a.y * b.y}; }
 inline uint32_t smem_u32(const void* p) { return (uint32_t)(uintptr_t)p; }
 struct ProfScope { ProfScope(int, int, int, int, cudaStream_t) {} };
 }  // namespace lp

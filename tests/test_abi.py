@@ -34,7 +34,7 @@ def test_struct_layouts_match_header(tmp_path):
              "lp_dec_weights": _lib.DecWeights, "lp_gemm_desc": _lib.GemmDesc, "lp_tp_desc": _lib.TpDesc,
              "lp_profile_record": _lib.ProfileRecord, "lp_linear_desc": _lib.LinearDesc, "lp_window_attn_desc": _lib.WindowAttnDesc,
              "lp_mingru_desc": _lib.MinGRUDesc, "lp_retention_desc": _lib.RetentionDesc, "lp_latent_desc": _lib.LatentDesc,
-             "lp_mlstm_desc": _lib.MLSTMDesc}
+             "lp_mlstm_desc": _lib.MLSTMDesc, "lp_gla_desc": _lib.GlaDesc, "lp_hyper_desc": _lib.HyperDesc}
     lines = []
     for cname, ct in pairs.items():
         lines.append(f'printf("{cname} %zu\\n", sizeof({cname}));')
