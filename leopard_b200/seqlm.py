@@ -767,7 +767,7 @@ class SeqLMEngine:
         rows, states, summaries, looks, keep = [], [], [], [], 0
         self._cache_index, self._state_index, self._summary_index, self._shift_index, self._conv_index = {}, {}, {}, [], {}
         self._prev_index = {}          # the previous token's input of a WKV mixer
-        if cfg.streams > int(self.L.lp_hyper_max_streams()):
+        if cfg.streams and cfg.streams > int(self.L.lp_hyper_max_streams()):
             raise ValueError(f"{cfg.streams} streams are not built")
 
         def look_back(m):      # how far back a windowed or block-local layer reads (None: everything)
