@@ -569,12 +569,13 @@ def main():
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--workload", default="cfg3", choices=["cfg3", "cfg2", "cfg4", "cfg5", "seqlm", "ronelorn", "gavatar", "kamosun",
-                                                              "komazen"],
+                                                              "komazen", "bezizen"],
                     help="cfg3 (default) = the metric's configuration; cfg2 = 1 x 1344^2; cfg4 = Idefics2 8 x 980^2; cfg5 = SFT step; "
                          "seqlm = prefill / decode of the layer-list language models beside the Llama-style decoder at equal size; "
                          "ronelorn = the same for the Ronelorn layers beside the Zudalorn stack at equal size; gavatar = the same for the Gavatar layers; kamosun = the same for the Kamosun layers; "
-                         "komazen = the same for the Komazen layers beside the Zudalorn and Kamosun stacks")
-    ap.add_argument("--seqlm-sizes", default="", help="seqlm / ronelorn / gavatar / kamosun / komazen: comma-separated subset of w1024,w2048,w4096 (default: all three)")
+                         "komazen = the same for the Komazen layers beside the Zudalorn and Kamosun stacks; "
+                         "bezizen = the same for the Bezizen layers beside the Zudalorn and Komazen stacks")
+    ap.add_argument("--seqlm-sizes", default="", help="seqlm / ronelorn / gavatar / kamosun / komazen / bezizen: comma-separated subset of w1024,w2048,w4096 (default: all three)")
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--no-extras", action="store_true", help="skip the library / strong-scaling / decode / front-end legs")
     ap.add_argument("--quick", action="store_true", help="1 warm-up, timed loop only (for runs under ncu)")
@@ -604,6 +605,9 @@ def main():
     if args.workload == "komazen":
         from benchmarks import komazen_bench
         return komazen_bench.run(args)
+    if args.workload == "bezizen":
+        from benchmarks import bezizen_bench
+        return bezizen_bench.run(args)
     if args.workload in ("cfg4", "cfg5"):
         from benchmarks import other_workloads
         return other_workloads.run(args)
