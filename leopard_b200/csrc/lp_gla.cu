@@ -9,8 +9,8 @@
 //
 //   lp_gla     prompts, portions and one-token steps alike.  The recurrence runs in REGISTERS: a CTA per (piece of a request, head, tile of
 //              32, 64 or 128 state columns), a warp owns 16 rows of the tile, a lane 1, 2 or 4 of its columns; two rows share an
-//              instruction (packed fp32 multiply-adds).  Tokens are staged in shared memory 8 or 16 at a time (decays evaluated on the
-//              way in); the state updates of a stage need no synchronisation, the warps' partial read-outs meet in shared memory once
+//              instruction (packed fp32 multiply-adds).  Tokens are staged in shared memory 8 at a time, the next stage copied asynchronously
+//              while one computes; the state updates of a stage need no synchronisation, the warps' partial read-outs meet in shared memory once
 //              per stage, and there a warp per token closes the head: norm, gain, gate.
 //     one piece per request   (one-token steps, short portions, batches that fill the GPU): the state comes from the request's slot and
 //              goes back there.
@@ -20,6 +20,7 @@
 //              Products of decays are used as they are (at most 1), so no logarithm is taken and nothing overflows.
 //   A row's result is the token-by-token recurrence in every case, up to the grouping of the sums at a piece's start.
 //   Value heads wider than 128 columns take several column tiles; their outputs go through a buffer and lp_gla's finish kernel.
+#include <cuda_pipeline.h>
 #include "lp_host.h"
 #include "../../include/leopard_b200.h"
 
@@ -54,31 +55,33 @@ struct GlaBatch {
 
 __device__ __forceinline__ float gla_decay(int kind, float e, float z) {
   if (kind == LP_GLA_DECAY_DOUBLE_EXP) return expf(-expf(z));
-  return expf(-e * (log1pf(expf(-fabsf(z))) + fmaxf(-z, 0.f)));      // sigmoid(z)^e = exp(-e softplus(-z))
+  // sigmoid(z)^e = exp(-e softplus(-z)); an absolute error of the logarithm is a relative one of the decay, so log(1 + x) serves
+  return expf(-e * (logf(1.0f + expf(-fabsf(z))) + fmaxf(-z, 0.f)));
 }
 
-// the decay of channel d of head h at `row`; without z it is made here from the low-rank vector t of the row
-__device__ __forceinline__ float gla_row_decay(const GlaArgs& a, long long row, int h, int d) {
-  const int n = h * a.dim + d;
-  float z;
-  if (a.z != nullptr) {
-    z = a.z[row * a.ldz + n];
-  } else {
-    z = a.z_bias != nullptr ? a.z_bias[n] : 0.f;
-    const float* t = a.t + row * a.ldt;
-    const bf16* w = a.w2 + (long long)n * a.ldw2;
-    for (int i = 0; i < a.rank; ++i) z = fmaf(__bfloat162float(w[i]), a.t_tanh ? tanhf(t[i]) : t[i], z);
+// the pre-activation of decay n of a row from the row's low-rank vector (t: activated when `active`)
+__device__ __forceinline__ float gla_low_rank(const GlaArgs& a, const float* t, bool active, int n) {
+  float z = a.z_bias != nullptr ? a.z_bias[n] : 0.f;
+  const bf16* w = a.w2 + (long long)n * a.ldw2;
+  int i = 0;
+  if (active && ((reinterpret_cast<uintptr_t>(w) & 15) == 0)) {      // eight factors a read
+    for (; i + 8 <= a.rank; i += 8) {
+      const uint4 u = *reinterpret_cast<const uint4*>(w + i);
+      const unsigned f[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        z = fmaf(__uint_as_float(f[j] << 16), t[i + 2 * j], z);
+        z = fmaf(__uint_as_float(f[j] & 0xffff0000u), t[i + 2 * j + 1], z);
+      }
+    }
   }
-  return gla_decay(a.decay, a.decay_exp, z);
+  for (; i < a.rank; ++i) z = fmaf(__bfloat162float(w[i]), active || !a.t_tanh ? t[i] : tanhf(t[i]), z);
+  return z;
 }
 
-__device__ __forceinline__ float gla_close(const GlaArgs& a, long long row, int h, int c, float o, float rinv) {
-  float v = o * rinv;
-  if (a.out_gain != nullptr) v *= a.out_gain[h * a.gain_stride + c];
-  if (a.gate != nullptr) {
-    const float g = a.gate[row * a.ldg + h * a.vdim + c];
-    v *= g / (1.0f + expf(-g));
-  }
+__device__ __forceinline__ float gla_close(float o, float rinv, float gain, const float* gate) {
+  float v = o * rinv * gain;
+  if (gate != nullptr) v *= __fdividef(*gate, 1.0f + expf(-*gate));
   return v;
 }
 __device__ __forceinline__ void gla_store(const GlaArgs& a, long long row, int h, int c, float v) {
@@ -87,17 +90,33 @@ __device__ __forceinline__ void gla_store(const GlaArgs& a, long long row, int h
   else reinterpret_cast<bf16*>(a.out)[at] = __float2bfloat16(v);
 }
 
-template <int CPL> struct GlaTile {
-  static constexpr int COLS = 32 * CPL, TOK = CPL == 4 ? 8 : 16;
-};
+constexpr int GLA_TOK = 8;              // tokens a stage
+
+// One operand of a stage: `n` floats of each of nt tokens (src_ld apart) into rows of dst, by all threads of the CTA; a thread's place (token
+// t, column c) in the stage is the caller's, `t_step` tokens further on each turn.
+__device__ __forceinline__ void gla_fetch(float* dst, int dst_ld, const float* src, long long src_ld, int n, int nt, int t, int c, int t_step,
+                                          bool vec) {
+  if (c >= n) return;
+  for (; t < nt; t += t_step) {
+    const float* from = src + t * src_ld + c;
+    float* to = dst + t * dst_ld + c;
+    if (vec) {
+      __pipeline_memcpy_async(to, from, 16);
+    } else {
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+        if (c + i < n) __pipeline_memcpy_async(to + i, from + i, 4);
+    }
+  }
+}
 
 // OUT: read-outs, from the stored state (group 0: the request's slot; else the piece's start state in u).  !OUT: contribution and decay
-// product of the pieces that another piece follows.
-template <int CPL, bool OUT>
+// product of the pieces that another piece follows.  The operands of a stage are copied asynchronously while the stage before computes.
+template <int CPL, bool OUT, bool BONUS>
 __global__ void __launch_bounds__(GLA_MAX_WARPS * 32)
-gla_run_kernel(GlaArgs a, GlaBatch b) {
+gla_run_kernel(GlaArgs a, GlaBatch b, int vec) {
   extern __shared__ float dyn_smem[];
-  constexpr int COLS = GlaTile<CPL>::COLS, TOK = GlaTile<CPL>::TOK;
+  constexpr int COLS = 32 * CPL, TOK = GLA_TOK;
   const int h = blockIdx.y, col0 = blockIdx.z * COLS;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, NW = blockDim.x >> 5, dpad = NW * GLA_ROWS;
   int s, row0, len;
@@ -117,12 +136,32 @@ gla_run_kernel(GlaArgs a, GlaBatch b) {
     row0 = b.chunk_row0[c];
     len = b.chunk_row0[c_last] + b.chunk_len[c_last] - row0;
   }
-  float* k_s = dyn_smem;                        // [TOK][dpad], zero beyond dim
-  float* w_s = k_s + TOK * dpad;                // [TOK][dpad] decays
-  float* v_s = w_s + TOK * dpad;                // [TOK][COLS]
-  float* q_s = v_s + TOK * COLS;                // OUT: [TOK][dpad]
-  float* red_s = q_s + (OUT ? TOK * dpad : 0);  // OUT: [TOK][NW][COLS] partial read-outs; else [2][dpad] partial decay products
+  // two stages of [k | z, turned into decays | v | (OUT) q | (OUT) gate], zero beyond dim and vdim
+  const int part = TOK * dpad, stage = (OUT ? 3 : 2) * part + (OUT ? 2 : 1) * TOK * COLS;
+  float* red_s = dyn_smem + 2 * stage;          // OUT: [TOK][NW][COLS] partial read-outs; else [2][dpad] partial decay products
   float* bon_s = red_s + TOK * NW * COLS;       // OUT: [TOK] sum_d bonus_d q_d k_d
+  const int cols = a.vdim - col0 < COLS ? a.vdim - col0 : COLS;
+  const bool gated = OUT && a.gate != nullptr && b.raw == nullptr;
+  if (a.dim < dpad || cols < COLS)
+    for (int i = tid; i < 2 * stage; i += blockDim.x) dyn_smem[i] = 0.f;
+  if (a.dim < dpad || cols < COLS) __syncthreads();
+  // four columns a thread: the 2 dpad threads cover 8 tokens of dpad channels at once, and a tile's columns in 32 NW / (COLS / 4) tokens a turn
+  const int f_t = tid / (dpad >> 2), f_c = tid % (dpad >> 2) * 4;
+  const int v_t = tid / (COLS / 4), v_c = tid % (COLS / 4) * 4, v_step = NW * 32 / (COLS / 4);
+  auto fetch = [&](int t0, int buf) {
+    const int nt = len - t0 < TOK ? len - t0 : TOK;
+    float* p = dyn_smem + buf * stage;
+    const long long row = row0 + t0;
+    gla_fetch(p, dpad, a.k + row * a.ldk + h * a.dim, a.ldk, a.dim, nt, f_t, f_c, TOK, vec);
+    if (a.z != nullptr) gla_fetch(p + part, dpad, a.z + row * a.ldz + h * a.dim, a.ldz, a.dim, nt, f_t, f_c, TOK, vec);
+    p += 2 * part;
+    gla_fetch(p, COLS, a.v + row * a.ldv + h * a.vdim + col0, a.ldv, cols, nt, v_t, v_c, v_step, vec);
+    p += TOK * COLS;
+    if (OUT) gla_fetch(p, dpad, a.q + row * a.ldq + h * a.dim, a.ldq, a.dim, nt, f_t, f_c, TOK, vec);
+    if (gated) gla_fetch(p + part, COLS, a.gate + row * a.ldg + h * a.vdim + col0, a.ldg, cols, nt, v_t, v_c, v_step, vec);
+    __pipeline_commit();
+  };
+  fetch(0, 0);
   const long long hs = (long long)a.dim * a.vdim;
   float* slot = a.state + (long long)b.seq_slot[s] * a.slot_stride + h * hs;
   float* piece = b.group ? b.u + ((long long)blockIdx.x * a.heads + h) * hs : nullptr;
@@ -138,30 +177,47 @@ gla_run_kernel(GlaArgs a, GlaBatch b) {
       S[rr][c].x = (stored && d < a.dim && y < a.vdim) ? src[(long long)d * a.vdim + y] : 0.f;
       S[rr][c].y = (stored && d + 1 < a.dim && y < a.vdim) ? src[(long long)(d + 1) * a.vdim + y] : 0.f;
     }
-  // a thread stages one channel d of every other token (the CTA has two threads per channel)
+  // without z the decays come from the low-rank vectors; a lone token's is activated once, ahead of its use
+  const bool low = a.z == nullptr, lone = low && len == 1 && OUT && a.rank <= TOK * NW * COLS;
+  if (lone)
+    for (int i = tid; i < a.rank; i += blockDim.x) {
+      const float t = a.t[row0 * a.ldt + i];
+      red_s[i] = a.t_tanh ? tanhf(t) : t;
+    }
+  // a thread turns one channel's pre-activations into decays, every other token's (the CTA has two threads per channel)
   const int my_d = tid % dpad, my_t = tid / dpad;
-  const bool live_d = my_d < a.dim;
   float prod = 1.f;
-  const float* kp = a.k + h * a.dim + my_d;
-  const float* qp = a.q + h * a.dim + my_d;
-  for (int t0 = 0; t0 < len; t0 += TOK) {
+  float gain[CPL];
+#pragma unroll
+  for (int c = 0; c < CPL; ++c) {
+    const int y = lane + 32 * c;
+    gain[c] = OUT && a.out_gain != nullptr && b.raw == nullptr && y < a.vdim ? a.out_gain[h * a.gain_stride + y] : 1.0f;
+  }
+  for (int t0 = 0, buf = 0; t0 < len; t0 += TOK, buf ^= 1) {
     const int nt = len - t0 < TOK ? len - t0 : TOK;
-    __syncthreads();      // the previous stage has been read
-#pragma unroll 4
-    for (int t = my_t; t < nt; t += 2) {
-      const long long row = row0 + t0 + t;
-      const float w = live_d ? gla_row_decay(a, row, h, my_d) : 1.f;
-      k_s[t * dpad + my_d] = live_d ? kp[row * a.ldk] : 0.f;
-      w_s[t * dpad + my_d] = w;
-      if (OUT) q_s[t * dpad + my_d] = live_d ? qp[row * a.ldq] * a.q_scale : 0.f;
-      else prod *= w;
+    __pipeline_wait_prior(0);
+    __syncthreads();      // this stage has arrived, the one before has been read
+    if (t0 + TOK < len) fetch(t0 + TOK, buf ^ 1);
+    const float* k_s = dyn_smem + buf * stage;
+    float* w_s = dyn_smem + buf * stage + part;
+    const float* v_s = w_s + part;
+    const float* q_s = v_s + TOK * COLS;
+    const float* g_s = q_s + part;
+    if (my_d < a.dim) {
+#pragma unroll
+      for (int j = 0; j < TOK / 2; ++j) {
+        const int t = my_t + 2 * j;
+        if (t < nt) {
+          float z;
+          if (!low) z = w_s[t * dpad + my_d];
+          else z = gla_low_rank(a, lone ? red_s : a.t + (row0 + t0 + t) * a.ldt, lone, h * a.dim + my_d);
+          const float w = gla_decay(a.decay, a.decay_exp, z);
+          w_s[t * dpad + my_d] = w;
+          if (!OUT) prod *= w;
+        }
+      }
     }
-    for (int i = tid; i < nt * COLS; i += blockDim.x) {
-      const int t = i / COLS, y = col0 + i % COLS;
-      v_s[i] = y < a.vdim ? a.v[(row0 + t0 + t) * a.ldv + h * a.vdim + y] : 0.f;
-    }
-    __syncthreads();
-    if (OUT && a.bonus != nullptr) {      // a warp per token; read after the next barrier
+    if (BONUS) {      // a warp per token; read after the next barrier but one
       for (int t = warp; t < nt; t += NW) {
         float acc = 0.f;
         for (int d = lane; d < a.dim; d += 32) acc = fmaf(a.bonus[h * a.dim + d] * q_s[t * dpad + d], k_s[t * dpad + d], acc);
@@ -170,7 +226,8 @@ gla_run_kernel(GlaArgs a, GlaBatch b) {
         if (lane == 0) bon_s[t] = acc;
       }
     }
-#pragma unroll 2
+    __syncthreads();
+#pragma unroll(CPL == 4 ? 2 : 1)
     for (int t = 0; t < nt; ++t) {
       float2 vv[CPL], acc[CPL];
 #pragma unroll
@@ -196,9 +253,9 @@ gla_run_kernel(GlaArgs a, GlaBatch b) {
 #pragma unroll
           for (int c = 0; c < CPL; ++c) {
             float2& st = S[2 * r4 + half][c];
-            if (OUT && a.bonus != nullptr) acc[c] = fma2(st, q2, acc[c]);      // the state before this token
+            if (OUT && BONUS) acc[c] = fma2(st, q2, acc[c]);      // the state before this token
             st = fma2(w2, st, mul2(k2, vv[c]));
-            if (OUT && a.bonus == nullptr) acc[c] = fma2(st, q2, acc[c]);
+            if (OUT && !BONUS) acc[c] = fma2(st, q2, acc[c]);
           }
         }
       }
@@ -214,10 +271,11 @@ gla_run_kernel(GlaArgs a, GlaBatch b) {
         float o[CPL], ss = 0.f;
 #pragma unroll
         for (int c = 0; c < CPL; ++c) {
-          float x = a.bonus != nullptr ? bon_s[t] * v_s[t * COLS + lane + 32 * c] : 0.f;
+          float x = BONUS ? bon_s[t] * v_s[t * COLS + lane + 32 * c] : 0.f;
+#pragma unroll 4
           for (int y = 0; y < NW; ++y) x += red_s[(t * NW + y) * COLS + lane + 32 * c];
-          o[c] = x;
-          ss = fmaf(x, x, ss);      // columns past vdim are zero
+          o[c] = x * a.q_scale;
+          ss = fmaf(o[c], o[c], ss);      // columns past vdim are zero
         }
         if (b.raw != nullptr) {
 #pragma unroll
@@ -233,7 +291,7 @@ gla_run_kernel(GlaArgs a, GlaBatch b) {
 #pragma unroll
         for (int c = 0; c < CPL; ++c) {
           const int y = lane + 32 * c;
-          if (y < a.vdim) gla_store(a, row, h, y, gla_close(a, row, h, y, o[c], rinv));
+          if (y < a.vdim) gla_store(a, row, h, y, gla_close(o[c], rinv, gain[c], gated ? g_s + t * COLS + y : nullptr));
         }
       }
     }
@@ -241,7 +299,8 @@ gla_run_kernel(GlaArgs a, GlaBatch b) {
   if (!OUT) {      // the product of the piece's decays: two partial products per channel
     red_s[my_t * dpad + my_d] = prod;
     __syncthreads();
-    if (blockIdx.z == 0 && my_t == 0 && live_d) b.p[((long long)blockIdx.x * a.heads + h) * a.dim + my_d] = red_s[my_d] * red_s[dpad + my_d];
+    if (blockIdx.z == 0 && my_t == 0 && my_d < a.dim)
+      b.p[((long long)blockIdx.x * a.heads + h) * a.dim + my_d] = red_s[my_d] * red_s[dpad + my_d];
   }
   if (!OUT || last) {
     float* dst = OUT ? slot : piece;
@@ -258,7 +317,7 @@ gla_run_kernel(GlaArgs a, GlaBatch b) {
 
 // one thread per state element of a (request, head): u[piece] <- state at the piece's start.  The pieces' contributions are loaded
 // several at a time (independent loads) ahead of the dependent multiply-adds.
-constexpr int GLA_SCAN_THREADS = 256, GLA_SCAN_BATCH = 8;
+constexpr int GLA_SCAN_THREADS = 256, GLA_SCAN_BATCH = 16;
 __global__ void __launch_bounds__(GLA_SCAN_THREADS)
 gla_scan_kernel(GlaArgs a, GlaBatch b) {
   const int s = blockIdx.x, h = blockIdx.y;
@@ -304,7 +363,9 @@ gla_finish_kernel(GlaArgs a, int R, const float* __restrict__ raw) {
 #pragma unroll
   for (int m = 16; m > 0; m >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, m);
   const float rinv = 1.0f / sqrtf(ss / (float)a.vdim + a.eps);
-  for (int c = lane; c < a.vdim; c += 32) gla_store(a, row, h, c, gla_close(a, row, h, c, o[c], rinv));
+  for (int c = lane; c < a.vdim; c += 32) 
+    gla_store(a, row, h, c, gla_close(o[c], rinv, a.out_gain != nullptr ? a.out_gain[h * a.gain_stride + c] : 1.0f,
+                                      a.gate != nullptr ? a.gate + (long long)row * a.ldg + h * a.vdim + c : nullptr));
 }
 
 // the operand of the low-rank decay product: act(t) as fp32, or split into two bf16 values hi + lo side by side (a product with the
@@ -327,38 +388,54 @@ __global__ void lowrank_operand_kernel(const float* __restrict__ t, long long ld
 
 template <int CPL>
 static size_t gla_smem_bytes(int warps, bool out) {
-  constexpr int COLS = GlaTile<CPL>::COLS, TOK = GlaTile<CPL>::TOK;
+  constexpr int COLS = 32 * CPL;
   const size_t dpad = (size_t)warps * GLA_ROWS;
-  return (2 * TOK * dpad + TOK * COLS + (out ? TOK * dpad + (size_t)TOK * warps * COLS + TOK : 2 * dpad)) * sizeof(float);
+  const size_t stage = (out ? 3 : 2) * GLA_TOK * dpad + (out ? 2 : 1) * GLA_TOK * COLS;
+  return (2 * stage + (out ? (size_t)GLA_TOK * warps * COLS + GLA_TOK : 2 * dpad)) * sizeof(float);
 }
 
-template <int CPL, bool OUT>
-static int launch_gla_run(const GlaArgs& a, const GlaBatch& b, int pieces, cudaStream_t stream) {
+template <int CPL, bool OUT, bool BONUS>
+static int launch_gla_run(const GlaArgs& a, const GlaBatch& b, int pieces, int vec, cudaStream_t stream) {
   const int warps = (a.dim + GLA_ROWS - 1) / GLA_ROWS;
   const size_t smem = gla_smem_bytes<CPL>(warps, OUT);
   static size_t have = 48 * 1024;      // raised once per instantiation, and only for head sizes that need it
   if (smem > have) {
-    LP_CHECK_CUDA(cudaFuncSetAttribute(gla_run_kernel<CPL, OUT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 120 * 1024));
-    have = 120 * 1024;
+    LP_CHECK_CUDA(cudaFuncSetAttribute(gla_run_kernel<CPL, OUT, BONUS>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024));
+    have = 160 * 1024;
   }
-  const dim3 grid(pieces, a.heads, (a.vdim + GlaTile<CPL>::COLS - 1) / GlaTile<CPL>::COLS);
-  gla_run_kernel<CPL, OUT><<<grid, warps * 32, smem, stream>>>(a, b);
+  const dim3 grid(pieces, a.heads, (a.vdim + 32 * CPL - 1) / (32 * CPL));
+  gla_run_kernel<CPL, OUT, BONUS><<<grid, warps * 32, smem, stream>>>(a, b, vec);
   LP_CHECK_CUDA(cudaGetLastError());
   return 0;
 }
 
 template <int CPL>
-static int launch_gla(const GlaArgs& a, GlaBatch b, int n_seqs, int n_chunks, cudaStream_t stream) {
+static int launch_gla_out(const GlaArgs& a, const GlaBatch& b, int pieces, int vec, cudaStream_t stream) {
+  if (a.bonus != nullptr) return launch_gla_run<CPL, true, true>(a, b, pieces, vec, stream);
+  return launch_gla_run<CPL, true, false>(a, b, pieces, vec, stream);
+}
+
+template <int CPL>
+static int launch_gla(const GlaArgs& a, GlaBatch b, int n_seqs, int n_chunks, int vec, cudaStream_t stream) {
   if (b.group == 0) {
     note_launch();
-    return launch_gla_run<CPL, true>(a, b, n_seqs, stream);
+    return launch_gla_out<CPL>(a, b, n_seqs, vec, stream);
   }
-  if (int rc = launch_gla_run<CPL, false>(a, b, n_chunks, stream)) return rc;
+  if (int rc = launch_gla_run<CPL, false, false>(a, b, n_chunks, vec, stream)) return rc;
   const long long hs = (long long)a.dim * a.vdim;
   gla_scan_kernel<<<dim3(n_seqs, a.heads, (unsigned)((hs + GLA_SCAN_THREADS - 1) / GLA_SCAN_THREADS)), GLA_SCAN_THREADS, 0, stream>>>(a, b);
   LP_CHECK_CUDA(cudaGetLastError());
   note_launch(3);
-  return launch_gla_run<CPL, true>(a, b, n_chunks, stream);
+  return launch_gla_out<CPL>(a, b, n_chunks, vec, stream);
+}
+
+// 16-byte copies need every operand's base and row stride, and the heads inside a row, on 16-byte boundaries
+static bool gla_vec(const GlaArgs& a) {
+  const void* bases[] = {a.q, a.k, a.v, a.z, a.gate};
+  for (const void* p : bases)
+    if (p != nullptr && (reinterpret_cast<uintptr_t>(p) & 15)) return false;
+  return a.dim % 4 == 0 && a.vdim % 4 == 0 && a.ldq % 4 == 0 && a.ldk % 4 == 0 && a.ldv % 4 == 0 && (a.z == nullptr || a.ldz % 4 == 0) &&
+         (a.gate == nullptr || a.ldg % 4 == 0);
 }
 
 static int gla_col_tiles(int vdim) { return (vdim + GLA_FUSED_COLS - 1) / GLA_FUSED_COLS; }
@@ -416,10 +493,11 @@ extern "C" int lp_gla(const lp_gla_desc* d, int n_seqs, int n_chunks, int R, int
   if (b.raw != nullptr) f += (size_t)R * d->heads * d->vdim;
   b.u = f;
   b.p = b.group ? f + (size_t)n_chunks * d->heads * d->dim * d->vdim : nullptr;
+  const int vec = gla_vec(a) ? 1 : 0;
   int rc;
-  if (d->vdim <= 32) rc = launch_gla<1>(a, b, n_seqs, n_chunks, stream);
-  else if (d->vdim <= 64) rc = launch_gla<2>(a, b, n_seqs, n_chunks, stream);
-  else rc = launch_gla<4>(a, b, n_seqs, n_chunks, stream);
+  if (d->vdim <= 32) rc = launch_gla<1>(a, b, n_seqs, n_chunks, vec, stream);
+  else if (d->vdim <= 64) rc = launch_gla<2>(a, b, n_seqs, n_chunks, vec, stream);
+  else rc = launch_gla<4>(a, b, n_seqs, n_chunks, vec, stream);
   if (rc != 0) return rc;
   if (b.raw != nullptr) {
     gla_finish_kernel<<<(R * d->heads + GLA_FIN_WARPS - 1) / GLA_FIN_WARPS, GLA_FIN_WARPS * 32, 0, stream>>>(a, R, b.raw);

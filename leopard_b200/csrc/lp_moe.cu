@@ -25,7 +25,7 @@ namespace lp {
 typedef __nv_bfloat16 bf16;
 
 constexpr int MOE_MAX_EXPERTS = 512, MOE_MAX_GROUPS = 64;
-constexpr int ROUTE_WARPS = 8;
+constexpr int ROUTE_WARPS = 8, ROUTE_WARPS_WIDE = 32, MOE_FEW_TOKENS = 296;      // few tokens (decoding) take wider CTAs
 
 // eight bf16 values of a 16-byte load -> fp32 (a bf16 is the upper half of an fp32)
 __device__ __forceinline__ void bf16x8_to_f32(const uint4& u, float* f) {
@@ -55,7 +55,7 @@ __device__ __forceinline__ void warp_best(float& v, int& i, int none) {
 // One CTA per token: the warps share out the router rows (and the gate row), 16-byte loads of the bf16 weights when the width
 // allows; then one warp makes the choice among the E scores.
 template <typename HT>
-__global__ void __launch_bounds__(ROUTE_WARPS * 32)
+__global__ void __launch_bounds__(ROUTE_WARPS_WIDE * 32)
 moe_route_kernel(const HT* __restrict__ h, long long ldh, int T, int D, const bf16* __restrict__ w_router, long long ldw, int E,
                  const float* __restrict__ correction, int n_groups, int keep_groups, int top, const bf16* __restrict__ w_gate,
                  int* __restrict__ idx_out, float* __restrict__ w_out, float* __restrict__ gate_out, int softmax_mode,
@@ -64,13 +64,13 @@ moe_route_kernel(const HT* __restrict__ h, long long ldh, int T, int D, const bf
   __shared__ float ch[MOE_MAX_EXPERTS];   // choice scores (minus infinity once taken or not eligible)
   __shared__ float gsc[MOE_MAX_GROUPS];   // group scores
   __shared__ int kept[MOE_MAX_GROUPS];
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n_warps = blockDim.x >> 5;
   const int t = blockIdx.x;
   if (t >= T) return;
   const HT* hr = h + (long long)t * ldh;
   const bool vec = (D % 8 == 0) && (ldw % 8 == 0) && ((reinterpret_cast<uintptr_t>(w_router) & 15) == 0) &&
                    (w_gate == nullptr || (reinterpret_cast<uintptr_t>(w_gate) & 15) == 0);
-  for (int e = warp; e <= E; e += ROUTE_WARPS) {
+  for (int e = warp; e <= E; e += n_warps) {
     if (e == E && w_gate == nullptr) break;
     const bf16* wr = e < E ? w_router + (long long)e * ldw : w_gate;
     float acc = 0.f;
@@ -213,6 +213,8 @@ __global__ void moe_combine_kernel(const float* __restrict__ y, long long ldy, c
   }
 }
 
+static int route_threads(int T, int E) { return 32 * (T > MOE_FEW_TOKENS || E < ROUTE_WARPS ? ROUTE_WARPS : E + 1 < ROUTE_WARPS_WIDE ? E + 1 : ROUTE_WARPS_WIDE); }
+
 }  // namespace lp
 
 using namespace lp;
@@ -232,11 +234,11 @@ extern "C" int lp_moe_route(const void* h, long long ldh, int h_fp32, int T, int
   if (T <= 0) return 0;
   const unsigned grid = (unsigned)T;
   if (h_fp32)
-    moe_route_kernel<float><<<grid, ROUTE_WARPS * 32, 0, stream>>>(reinterpret_cast<const float*>(h), ldh, T, D,
+    moe_route_kernel<float><<<grid, route_threads(T, E), 0, stream>>>(reinterpret_cast<const float*>(h), ldh, T, D,
         reinterpret_cast<const bf16*>(w_router), ldw, E, correction, n_groups, keep_groups, top, reinterpret_cast<const bf16*>(w_gate),
         idx_out, w_out, gate_out, 0, nullptr, 1.0f);
   else
-    moe_route_kernel<bf16><<<grid, ROUTE_WARPS * 32, 0, stream>>>(reinterpret_cast<const bf16*>(h), ldh, T, D,
+    moe_route_kernel<bf16><<<grid, route_threads(T, E), 0, stream>>>(reinterpret_cast<const bf16*>(h), ldh, T, D,
         reinterpret_cast<const bf16*>(w_router), ldw, E, correction, n_groups, keep_groups, top, reinterpret_cast<const bf16*>(w_gate),
         idx_out, w_out, gate_out, 0, nullptr, 1.0f);
   note_launch();
@@ -253,10 +255,10 @@ extern "C" int lp_moe_route_softmax(const void* h, long long ldh, int h_fp32, in
   if (T <= 0) return 0;
   const unsigned grid = (unsigned)T;
   if (h_fp32)
-    moe_route_kernel<float><<<grid, ROUTE_WARPS * 32, 0, stream>>>(reinterpret_cast<const float*>(h), ldh, T, D,
+    moe_route_kernel<float><<<grid, route_threads(T, E), 0, stream>>>(reinterpret_cast<const float*>(h), ldh, T, D,
         reinterpret_cast<const bf16*>(w_router), ldw, E, nullptr, 1, 1, top, nullptr, idx_out, w_out, nullptr, 1, logit_bias, 1.0f);
   else
-    moe_route_kernel<bf16><<<grid, ROUTE_WARPS * 32, 0, stream>>>(reinterpret_cast<const bf16*>(h), ldh, T, D,
+    moe_route_kernel<bf16><<<grid, route_threads(T, E), 0, stream>>>(reinterpret_cast<const bf16*>(h), ldh, T, D,
         reinterpret_cast<const bf16*>(w_router), ldw, E, nullptr, 1, 1, top, nullptr, idx_out, w_out, nullptr, 1, logit_bias, 1.0f);
   note_launch();
   LP_CHECK_CUDA(cudaGetLastError());
@@ -272,10 +274,10 @@ extern "C" int lp_moe_route_sigmoid(const void* h, long long ldh, int h_fp32, in
   if (T <= 0) return 0;
   const unsigned grid = (unsigned)T;
   if (h_fp32)
-    moe_route_kernel<float><<<grid, ROUTE_WARPS * 32, 0, stream>>>(reinterpret_cast<const float*>(h), ldh, T, D,
+    moe_route_kernel<float><<<grid, route_threads(T, E), 0, stream>>>(reinterpret_cast<const float*>(h), ldh, T, D,
         reinterpret_cast<const bf16*>(w_router), ldw, E, nullptr, 1, 1, top, nullptr, idx_out, w_out, nullptr, 2, nullptr, 1.0f);
   else
-    moe_route_kernel<bf16><<<grid, ROUTE_WARPS * 32, 0, stream>>>(reinterpret_cast<const bf16*>(h), ldh, T, D,
+    moe_route_kernel<bf16><<<grid, route_threads(T, E), 0, stream>>>(reinterpret_cast<const bf16*>(h), ldh, T, D,
         reinterpret_cast<const bf16*>(w_router), ldw, E, nullptr, 1, 1, top, nullptr, idx_out, w_out, nullptr, 2, nullptr, 1.0f);
   note_launch();
   LP_CHECK_CUDA(cudaGetLastError());
@@ -296,10 +298,10 @@ extern "C" int lp_moe_route_group_softmax(const void* h, long long ldh, int h_fp
   if (T <= 0) return 0;
   const unsigned grid = (unsigned)T;
   if (h_fp32)
-    moe_route_kernel<float><<<grid, ROUTE_WARPS * 32, 0, stream>>>(reinterpret_cast<const float*>(h), ldh, T, D,
+    moe_route_kernel<float><<<grid, route_threads(T, E), 0, stream>>>(reinterpret_cast<const float*>(h), ldh, T, D,
         reinterpret_cast<const bf16*>(w_router), ldw, E, nullptr, n_groups, keep_groups, top, nullptr, idx_out, w_out, nullptr, 3, nullptr, w_scale);
   else
-    moe_route_kernel<bf16><<<grid, ROUTE_WARPS * 32, 0, stream>>>(reinterpret_cast<const bf16*>(h), ldh, T, D,
+    moe_route_kernel<bf16><<<grid, route_threads(T, E), 0, stream>>>(reinterpret_cast<const bf16*>(h), ldh, T, D,
         reinterpret_cast<const bf16*>(w_router), ldw, E, nullptr, n_groups, keep_groups, top, nullptr, idx_out, w_out, nullptr, 3, nullptr, w_scale);
   note_launch();
   LP_CHECK_CUDA(cudaGetLastError());
@@ -339,7 +341,8 @@ extern "C" int lp_moe_combine(const float* y, long long ldy, const int* pair_row
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
   LP_REQUIRE(y != nullptr && pair_row != nullptr && out != nullptr, "lp_moe_combine: null operand");
   if (T <= 0) return 0;
-  moe_combine_kernel<<<T, 128, 0, stream>>>(y, ldy, pair_row, w, top, shared, lds, gate, out, ldo, T, D);
+  const int threads = T > MOE_FEW_TOKENS || D < 512 ? 128 : D < 1024 ? 256 : 1024;
+  moe_combine_kernel<<<T, threads, 0, stream>>>(y, ldy, pair_row, w, top, shared, lds, gate, out, ldo, T, D);
   note_launch();
   LP_CHECK_CUDA(cudaGetLastError());
   return 0;

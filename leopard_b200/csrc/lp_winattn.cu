@@ -114,8 +114,8 @@ __device__ __forceinline__ const float* win_visible_row(const WinArgs& a, const 
   return win_token_row(a, seq, v.lo + (t - v.n_keep - v.n_blocks));
 }
 
-constexpr int WIN_PREP_THREADS = 128;
-__global__ void __launch_bounds__(WIN_PREP_THREADS)
+constexpr int WIN_PREP_THREADS = 128, WIN_PREP_WIDE = 1024;      // few rows (decoding) take the wide CTA
+__global__ void __launch_bounds__(WIN_PREP_WIDE)
 window_attn_prep_kernel(WinArgs a, int R, const int* __restrict__ row_seq, const int* __restrict__ row_pos) {
   extern __shared__ float dyn_smem[];
   float* s_ss = dyn_smem;      // [heads + kv_heads] sums of squares, then the two totals
@@ -1143,6 +1143,7 @@ static int fill_win(WinArgs& a, const lp_window_attn_desc* d, bool need_q) {
 }
 
 constexpr int WIN_MAX_DIM = 256;
+constexpr int WIN_PREP_ROWS = 296;      // up to two rows a multiprocessor
 constexpr int WIN_SPLIT_ROWS = 16;      // up to this many rows (decoding) a CTA has 8 warps, else 4
 
 static size_t win_smem_floats(int qh, int w, int dim, int vdim) {
@@ -1204,7 +1205,9 @@ extern "C" int lp_window_attn_prep(const lp_window_attn_desc* d, int R, const in
   if (R <= 0) return 0;
   const size_t smem = (size_t)(d->heads + 2 * d->kv_heads + 2) * sizeof(float);
   LP_REQUIRE(smem <= 48 * 1024, "lp_window_attn_prep: too many heads");
-  window_attn_prep_kernel<<<R, WIN_PREP_THREADS, smem, stream>>>(a, R, row_seq, row_pos);
+  // one row is a CTA: with few rows it should not walk its elements 128 at a time
+  const int wide = d->heads * d->dim >= WIN_PREP_WIDE ? WIN_PREP_WIDE : 256;
+  window_attn_prep_kernel<<<R, R <= WIN_PREP_ROWS ? wide : WIN_PREP_THREADS, smem, stream>>>(a, R, row_seq, row_pos);
   note_launch();
   LP_CHECK_CUDA(cudaGetLastError());
   return 0;

@@ -796,7 +796,7 @@ class SeqLMEngine:
             elif isinstance(m, WindowAttentionConfig):
                 ci = len(rows)
                 rows.append(m.kv_heads * (m.dim + (0 if m.values_are_keys else m.vdim)))
-                if m.qk_conv > int(self.L.lp_causal_conv_max_taps()):
+                if m.qk_conv and m.qk_conv > int(self.L.lp_causal_conv_max_taps()):
                     raise ValueError(f"layer {key}: a convolution of {m.qk_conv} taps is not built")
                 if m.qk_conv > 1:      # the last taps - 1 projected queries and keys
                     self._conv_index[(key, "qk")] = len(states)
